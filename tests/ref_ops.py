@@ -59,8 +59,14 @@ def _checked(ids, bound: int, bit: int):
     return ids
 
 
-def embed(ids, table, scale=1.0):
-    return _f(table[_checked(ids.long(), table.shape[0], 2)]) * scale
+def embed(ids, table, scale=1.0, positions=None, base=10000.0):
+    out = _f(table[_checked(ids.long(), table.shape[0], 2)]) * scale
+    if positions is not None:                # sines in the even, cosines in the odd entries
+        W = table.shape[1]
+        angle = positions.double()[:, None] * float(base) ** (-2.0 * torch.arange((W + 1) // 2, dtype=torch.float64, device=table.device) / W)
+        vec = torch.stack([torch.sin(angle), torch.cos(angle)], dim=-1).reshape(len(positions), -1)[:, :W]
+        out = out + vec.float()
+    return out
 
 
 def _normed(delta, gamma, eps):
@@ -320,6 +326,8 @@ def activation(x, kind):
         y = _silu(v)
     elif kind == "relu":
         y = torch.relu(v)
+    elif kind == "relu2":
+        y = torch.relu(v) ** 2
     else:
         raise KeyError(kind)
     return y.to(x.dtype)
@@ -595,14 +603,18 @@ def rmsnorm_rows(x, w, eps):
 
 
 def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on="input", score="sigmoid", act="silu", limit=0.0,
-                   alpha=1.702):
+                   alpha=1.702, router_bias=None, unit=None, unit_gated=False):
     """Every row to the `top` experts with the largest sigmoid(x . w_router^T); the scores weigh the experts' inputs
-    or outputs; w_gate_up [E, 2F, W] (gate rows, then up rows), w_down [E, W, F]."""
+    or outputs; w_gate_up [E, 2F, W] (gate rows, then up rows; [E, F, W] for "relu2"), w_down [E, W, F]."""
     N, W = x.shape
-    E, F = w_gate_up.shape[0], w_gate_up.shape[1] // 2
+    E, F = w_gate_up.shape[0], w_gate_up.shape[1] // (1 if act == "relu2" else 2)
     z = _f(x) @ _f(w_router).t()
-    s = torch.softmax(z, dim=-1) if score == "softmax" else torch.sigmoid(z)
+    gate = torch.sigmoid(z[:, E:]) if unit_gated else None
+    z = z[:, :E] if router_bias is None else z[:, :E] + router_bias
+    s = torch.softmax(z, dim=-1) if score == "softmax" else z if score == "chosen" else torch.sigmoid(z)
     val, idx = torch.topk(s, int(top), dim=-1)
+    if score == "chosen":
+        val = torch.softmax(val, dim=-1)
     if renorm:
         val = val / (val.sum(-1, keepdim=True) + 1e-20)
     out = torch.zeros((N, W), dtype=torch.float32, device=x.device)
@@ -611,14 +623,50 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
             e, w = int(idx[n, k]), val[n, k]
             xin = (_f(x[n]) * w).to(x.dtype) if weight_on == "input" else x[n]
             gu = _f(xin) @ _f(w_gate_up[e]).t()
-            if act == "clamped":
+            if act == "relu2":
+                hid = (torch.relu(gu) ** 2).to(x.dtype)
+            elif act == "clamped":
                 g, u = torch.clamp(gu[:F], max=limit), torch.clamp(gu[F:], min=-limit, max=limit)
                 hid = (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(x.dtype)
             else:
                 hid = (_silu(gu[:F]) * gu[F:]).to(x.dtype)
             y = _f(hid) @ _f(w_down[e]).t()
             out[n] += y if weight_on == "input" else y * w
+    if unit is not None:
+        out += _f(unit) if gate is None else gate * _f(unit)
     return out.to(x.dtype)
+
+
+def attention_difference(o, heads, vdim, cache_dim, lam, factor, eps):
+    """o [N, 2 * heads * cache_dim], a head's two maps side by side: factor * d / rms(d), d = o1 - lam * o2 over vdim."""
+    m = _f(o).reshape(o.shape[0], heads, 2, cache_dim)[..., :vdim]
+    return (factor * _rms(m[:, :, 0] - lam * m[:, :, 1], None, eps)).reshape(o.shape[0], heads * vdim).to(o.dtype)
+
+
+def mamba2(y, at, conv_w, conv_b, dt_bias, a_log, d_skip, norm_w, eps, norm_parts, state, conv_state, step, heads, groups, state_dim,
+           vdim, write_state=True, impl=None, precision=torch.float32):
+    """The state-space recurrence with one decay per head over the in-projection's rows y (columns `at`: z, x | B | C, dt);
+    state [slots, H, Ns, V], conv_state [slots, L - 1, channels].  `precision`: the type the recurrence is computed in."""
+    c = lambda t: t.to(precision)
+    N, H, G, Ns, V = y.shape[0], heads, groups, state_dim, vdim
+    I = H * V
+    z_at, xbc_at, dt_at = at
+    u = c(causal_conv(y[:, xbc_at:xbc_at + I + 2 * G * Ns], conv_w, conv_b, conv_state, step, True, write_state))
+    x = u[:, :I].reshape(N, H, V)
+    B, C = (t.reshape(N, G, Ns).repeat_interleave(H // G, dim=1) for t in (u[:, I:I + G * Ns], u[:, I + G * Ns:]))
+    d = torch.nn.functional.softplus(c(y[:, dt_at:dt_at + H]) + c(dt_bias), threshold=40.0)
+    keep = torch.exp(-torch.exp(c(a_log)) * d)
+    o = torch.zeros((N, H, V), dtype=precision, device=y.device)
+    for a, b, slot in _spans(step, state):
+        S = c(state[slot]).clone()
+        for t in range(a, b):
+            S = keep[t][:, None, None] * S + d[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
+            o[t] = torch.einsum("hnv,hn->hv", S, C[t]) + c(d_skip)[:, None] * x[t]
+        if write_state:
+            state[slot] = S.to(state.dtype)
+    g = o.reshape(N, I) * _silu(c(y[:, z_at:z_at + I]))
+    g = _rms(g.reshape(N, norm_parts, I // norm_parts), None, eps).reshape(N, I)
+    return (g * c(norm_w)).to(y.dtype)
 
 
 def act_mul(gu, ff_dim, kind):

@@ -50,12 +50,13 @@ ZAI_API int zai_silu_mul(void* out, const void* gu, int dtype, int N, int F, cud
     ZAI_DISPATCH(dtype, return launch_pdl(silu_mul_kernel<T>, dim3(blocks), dim3(threads), 0, stream, (T*)out, (const T*)gu, F, total));
 }
 
-// ---- an activation on its own:  0 exact (erf) GELU, 1 tanh GELU, 2 SiLU, 3 ReLU; computed in 32-bit
+// ---- an activation on its own:  0 exact (erf) GELU, 1 tanh GELU, 2 SiLU, 3 ReLU, 4 the square of ReLU; computed in 32-bit
 __device__ __forceinline__ float zai_activate(float v, int kind) {
     switch (kind) {
         case 0: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
         case 1: return 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
         case 2: return v / (1.f + expf(-v));
+        case 4: return fmaxf(v, 0.f) * fmaxf(v, 0.f);
         default: return fmaxf(v, 0.f);
     }
 }
@@ -74,7 +75,7 @@ __global__ void act_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, in
 ZAI_API int zai_act_mul(void* out, const void* gu, int dtype, int N, int F, int kind, cudaStream_t stream) {
     const size_t total = (size_t)N * F;
     if (total == 0) return ZAI_OK;
-    if (kind < 0 || kind > 3) return ZAI_BAD_SIZE;
+    if (kind < 0 || kind > 4) return ZAI_BAD_SIZE;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     ZAI_DISPATCH(dtype, return launch_pdl(act_mul_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)out, (const T*)gu, F, total, kind));
 }
@@ -106,7 +107,7 @@ __global__ void activation_bf16x8_kernel(bf16* __restrict__ out, const bf16* __r
 
 ZAI_API int zai_activation(void* out, const void* in, int dtype, int kind, long long total, cudaStream_t stream) {
     if (total <= 0) return ZAI_OK;
-    if (kind < 0 || kind > 3) return ZAI_BAD_SIZE;
+    if (kind < 0 || kind > 4) return ZAI_BAD_SIZE;
     const int threads = 256;
     if (dtype == ZAI_BF16 && (total & 7) == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(in)) & 15) == 0) {
         const size_t total8 = (size_t)total / 8;

@@ -86,6 +86,7 @@ struct SkinnyArgs {
     // the scaled sums
     int center;
     const float* beta_dot;
+    int plain_act;        // bfloat16 epilogue: 1: y = relu(.)^2, 0: as it is
 };
 
 __device__ __forceinline__ void cp_async16_zfill(void* smem, const void* gmem, bool valid) {
@@ -524,6 +525,10 @@ __global__ void __launch_bounds__(SG_WARPS * 32, 2) skinny_gemm_kernel(const Ski
                     if (row_lo >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.ldy + row_lo] = lo;
                     if (row_hi >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.ldy + row_hi] = hi;
                 } else {
+                    if (EPI == EPI_BF16 && a.plain_act) {
+                        lo = fmaxf(lo, 0.f) * fmaxf(lo, 0.f);
+                        hi = fmaxf(hi, 0.f) * fmaxf(hi, 0.f);
+                    }
                     if (row_lo >= 0) reinterpret_cast<bf16*>(a.y)[(size_t)tok * a.ldy + row_lo] = __float2bfloat16_rn(lo);
                     if (row_hi >= 0) reinterpret_cast<bf16*>(a.y)[(size_t)tok * a.ldy + row_hi] = __float2bfloat16_rn(hi);
                 }
@@ -886,9 +891,9 @@ static int skinny_run(SkinnyArgs& a, int epilogue, cudaStream_t stream) {
 static int skinny_gemm_run(void* y, const void* W, const void* x, const float* h, const void* delta,
                            const float* gamma, const int* row_idx, float* h_out, float eps, int M, int O, int K,
                            int epilogue, float glu_limit, float glu_slope, cudaStream_t stream, int center = 0,
-                           const float* beta_dot = nullptr) {
+                           const float* beta_dot = nullptr, int plain_act = 0) {
     if (epilogue == EPI_CONV || !zai_skinny_gemm_supports(M, O, K, epilogue, h != nullptr)) return ZAI_BAD_SIZE;
-    const int cs = (!h && (epilogue == EPI_BF16 || epilogue == EPI_F32)) ? splitk_cluster(K) : 0;
+    const int cs = (!h && !plain_act && (epilogue == EPI_BF16 || epilogue == EPI_F32)) ? splitk_cluster(K) : 0;
     if (cs) {
         SplitKArgs b = {};
         b.W = (const bf16*)W; b.x = (const bf16*)x; b.y = y; b.M = M; b.O = O; b.K = K;
@@ -907,6 +912,7 @@ static int skinny_gemm_run(void* y, const void* W, const void* x, const float* h
     a.glu_slope = glu_slope;
     a.center = center;
     a.beta_dot = beta_dot;
+    a.plain_act = plain_act;
     a.ldy = epilogue == EPI_SWIGLU ? O / 2 : O;
     if (epilogue == EPI_SWIGLU) {
         skinny_plan(a.F * 2, false, K, &a.n_tiles, &a.half_tiles, &a.tpc, &a.sk, &a.units);   // 8 gate + 8 up rows per tile
@@ -939,6 +945,12 @@ ZAI_API int zai_skinny_gemm_clamped_glu(void* y, const void* W, const void* x, c
                                         float limit, float slope, cudaStream_t stream) {
     if (limit == 0.f) return ZAI_BAD_SIZE;               // (limit < 0: the tanh-GELU gate, see the kernel's arguments)
     return skinny_gemm_run(y, W, x, h, delta, gamma, row_idx, h_out, eps, M, O, K, EPI_SWIGLU, limit, slope, stream);
+}
+
+// y = relu(x . W^T)^2, bfloat16 [M, O]; x or the norm of h as above.
+ZAI_API int zai_skinny_gemm_relu2(void* y, const void* W, const void* x, const float* h, const void* delta, const float* gamma,
+                                  const int* row_idx, float* h_out, float eps, int M, int O, int K, cudaStream_t stream) {
+    return skinny_gemm_run(y, W, x, h, delta, gamma, row_idx, h_out, eps, M, O, K, EPI_BF16, 0.f, 1.f, stream, 0, nullptr, 1);
 }
 
 // The short convolution's input projection with the convolution as its epilogue, for steps in which

@@ -44,6 +44,32 @@ __global__ void embed_bf16x8_kernel(float* __restrict__ out, const bf16* __restr
     }
 }
 
+// ... plus the sinusoidal vector of the row's position: entries 2i and 2i + 1 are sine and cosine of position * freq[i].  The
+// angle is a 64-bit product, brought into one turn in 64-bit; its sine and cosine are 32-bit.
+template <typename T>
+__global__ void embed_sinusoidal_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids, int H, int V,
+                                        float scale, const int* __restrict__ positions, const double* __restrict__ freq,
+                                        int* __restrict__ status) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = ids[t];
+    if ((unsigned)id >= (unsigned)V) {               // never read outside the table
+        if (threadIdx.x == 0) zai_raise(status, ZAI_ST_TOKEN);
+        id = 0;
+    }
+    const T* row = table + (size_t)id * H;
+    float* o = out + (size_t)t * H;
+    const double pos = (double)positions[t], turn = 6.283185307179586476925287;
+    for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
+        const double a = pos * freq[i];
+        float s, c;
+        sincosf((float)(a - rint(a / turn) * turn), &s, &c);
+        o[2 * i] = to_float(row[2 * i]) * scale + s;
+        if (2 * i + 1 < H) o[2 * i + 1] = to_float(row[2 * i + 1]) * scale + c;
+    }
+}
+
 // out[r] = h[rows[r]] (+ pending[rows[r]])
 template <typename T>
 __global__ void gather_add_kernel(float* __restrict__ out, const float* __restrict__ h,
@@ -95,6 +121,14 @@ ZAI_API int zai_embed(float* out, const void* table, int table_dtype, const int*
         return launch_pdl(embed_bf16x8_kernel, dim3(N), dim3(threads), 0, stream, out, (const bf16*)table, ids, H, V, scale, status);
     }
     ZAI_DISPATCH(table_dtype, return launch_pdl(embed_kernel<T>, dim3(N), dim3(256), 0, stream, out, (const T*)table, ids, H, V, scale, status));
+}
+
+// freq [(H + 1) / 2] in 64-bit
+ZAI_API int zai_embed_sinusoidal(float* out, const void* table, int table_dtype, const int* ids, int N, int H, int V, float scale,
+                                 const int* positions, const double* freq, int* status, cudaStream_t stream) {
+    if (N <= 0) return ZAI_OK;
+    ZAI_DISPATCH(table_dtype, return launch_pdl(embed_sinusoidal_kernel<T>, dim3(N), dim3(H >= 512 ? 256 : 128), 0, stream, out,
+                                                (const T*)table, ids, H, V, scale, positions, freq, status));
 }
 
 ZAI_API int zai_gather_add(float* out, const float* h, const void* pending, int pending_dtype, const int* rows,

@@ -37,6 +37,7 @@
 #define TC_SPIN_LIMIT 4000000
 
 enum { TC_EPI_BF16 = 0, TC_EPI_F32 = 1, TC_EPI_SWIGLU = 2,
+       TC_EPI_RELU2 = 4,        // bfloat16, the square of relu
        TC_EPI_F32_PAIR = 3 };   // (grouped products only) 32-bit results, two adjacent weight tiles against one token tile
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -255,6 +256,9 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tc_kernel(const __grid_consta
                             if (o + TC_BM < o_limit) reinterpret_cast<float*>(a.y)[(size_t)n * a.ldy + o + TC_BM] = __uint_as_float(u[j]);
                         } else if (EPI == TC_EPI_F32) {
                             reinterpret_cast<float*>(a.y)[(size_t)n * a.ldy + o] = v;
+                        } else if (EPI == TC_EPI_RELU2) {
+                            const float p = fmaxf(v, 0.f);
+                            reinterpret_cast<bf16*>(a.y)[(size_t)n * a.ldy + o] = __float2bfloat16_rn(p * p);
                         } else {
                             reinterpret_cast<bf16*>(a.y)[(size_t)n * a.ldy + o] = __float2bfloat16_rn(v);
                         }
@@ -375,14 +379,14 @@ ZAI_API int zai_gemm_tc(void* y, const void* W, const void* x, int* status, int 
 
 // Grouped products over rows sorted by group: x [n_tiles * 128, K]; W [groups, O, K]; token tile i (128 rows) takes the
 // matrix of group tile_group[i] (device memory; negative: the tile is skipped and its rows of y stay as they are).
-// Epilogues as above: y [n_tiles * 128, O] bfloat16 or 32-bit, or with SwiGLU [n_tiles * 128, O / 2].
+// Epilogues as above: y [n_tiles * 128, O] bfloat16 or 32-bit, or with SwiGLU [n_tiles * 128, O / 2]; 4: bfloat16 relu(.)^2.
 ZAI_API int zai_gemm_tc_grouped(void* y, const void* W, const void* x, const int* tile_group, int* status, int n_tiles, int groups,
                                 int O, int K, int epilogue, cudaStream_t stream) {
     if (n_tiles <= 0) return ZAI_OK;
     const long long rows = (long long)n_tiles * 128, w_rows = (long long)groups * O;
     const bool pair = epilogue == TC_EPI_F32_PAIR;
     if (pair) epilogue = TC_EPI_F32;
-    if (epilogue != TC_EPI_BF16 && epilogue != TC_EPI_F32 && epilogue != TC_EPI_SWIGLU) return ZAI_BAD_SIZE;
+    if (epilogue != TC_EPI_BF16 && epilogue != TC_EPI_F32 && epilogue != TC_EPI_SWIGLU && epilogue != TC_EPI_RELU2) return ZAI_BAD_SIZE;
     if (groups < 1 || rows > 0x7fffffff || w_rows > 0x7fffffff || !zai_gemm_tc_supports((int)rows, O, K, epilogue)) return ZAI_BAD_SIZE;
     if ((reinterpret_cast<uintptr_t>(W) & 15) || (reinterpret_cast<uintptr_t>(x) & 15) || !tile_group) return ZAI_BAD_SIZE;
     CUtensorMap mw, mx;
@@ -398,6 +402,7 @@ ZAI_API int zai_gemm_tc_grouped(void* y, const void* W, const void* x, const int
     a.tile_group = tile_group; a.group_rows = O;
     const int o_tiles = ((epilogue == TC_EPI_SWIGLU ? a.F : O) + TC_BM - 1) / TC_BM;
     if (epilogue == TC_EPI_BF16) return tc_launch<128, TC_EPI_BF16, 2>(mw, mx, a, o_tiles, stream);
+    if (epilogue == TC_EPI_RELU2) return tc_launch<128, TC_EPI_RELU2, 2>(mw, mx, a, o_tiles, stream);
     // two weight tiles a stage share the token tile (half the token tiles' traffic from L2 per product, as in the
     // gate/up product)
     if (pair && O > TC_BM) return tc_launch<128, TC_EPI_F32_PAIR, 2>(mw, mx, a, (O + 2 * TC_BM - 1) / (2 * TC_BM), stream);

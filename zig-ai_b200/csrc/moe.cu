@@ -1,9 +1,13 @@
 // A mixture of small gated feed-forwards: every row of the step goes to its `top` experts by router score.
 //
 //   z = x . Wr^T (32-bit),  s = sigmoid(z),  the `top` largest s choose the experts (ties: the lower index),
-//   weights w = s of the chosen (divided by their sum with `renorm`)
+//   weights w = s of the chosen (divided by their sum with `renorm`); or the logits themselves, z plus an optional bias,
+//   choose, and w = softmax over the chosen logits alone
 //   y = sum over the chosen e of  down_e( silu(gate_e(x_e)) * up_e(x_e) ),   x_e = w_e x   (`weight_on` input)
 //                                or of  w_e down_e( silu(gate_e(x)) * up_e(x) )             (`weight_on` output)
+//
+// The experts may also be units without a gate, down_e( act(up_e(x)) ), act the square of relu; and a unit that every row
+// passes beside its experts joins in the combine, weighed by the sigmoid of one more 32-bit product of the row.
 //
 // Five kernels, none of which tells the host anything (the step stays a fixed list of launches):
 //   * route: a block a row; the router's products summed in 32-bit in an order that depends on the width alone, the
@@ -56,11 +60,12 @@ __device__ __forceinline__ bool moe_rows_aligned(const T* p, size_t stride, int 
 }
 
 // ------------------------------------------------------------------------------------------------ route
+enum { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_LOGITS = 2 };          // what the scores are
 template <typename T>
 __global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ rank,
                                                         int* __restrict__ counts, const T* __restrict__ x, int x_stride,
                                                         const float* __restrict__ wr, int W, int E, int top, int renorm,
-                                                        int softmax) {
+                                                        int score, const float* __restrict__ bias, float* __restrict__ unit_gate) {
     extern __shared__ float sc[];                        // [E] scores
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_trigger();
@@ -68,7 +73,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, f
     const T* row = x + (size_t)t * x_stride;
     // (which of the two loops runs depends on the sizes and addresses alone, never on the other rows of the step)
     const bool vec = moe_rows_aligned(x, (size_t)x_stride, W) && (reinterpret_cast<uintptr_t>(wr) & 15) == 0;
-    for (int e = warp; e < E; e += 4) {
+    for (int e = warp; e < E + (unit_gate ? 1 : 0); e += 4) {
         const float* w = wr + (size_t)e * W;
         float acc = 0.f;
         if (vec) {
@@ -83,11 +88,14 @@ __global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, f
             for (int c = lane; c < W; c += 32) acc += to_float(row[c]) * w[c];
         }
         acc = warp_sum(acc);
-        if (lane == 0) sc[e] = softmax ? acc : 1.f / (1.f + expf(-acc));
+        if (lane == 0) {
+            if (e == E) unit_gate[t] = 1.f / (1.f + expf(-acc));         // (the row behind the router's: the unit beside the experts)
+            else sc[e] = score == MOE_SIGMOID ? 1.f / (1.f + expf(-acc)) : bias ? acc + bias[e] : acc;
+        }
     }
     __syncthreads();
     if (warp != 0) return;
-    if (softmax) {                                       // scores = softmax of the logits over all experts, in a fixed order
+    if (score == MOE_SOFTMAX) {                          // scores = softmax of the logits over all experts, in a fixed order
         float top_z = -INFINITY;
         for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, sc[e]);
         top_z = warp_max(top_z);
@@ -97,9 +105,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, f
         for (int e = lane; e < E; e += 32) sc[e] = expf(sc[e] - top_z) / total;
         __syncwarp();
     }
-    float sum = 0.f;
+    float sum = 0.f, mine = -INFINITY, first = 0.f;      // (`mine`: lane k keeps the k-th choice's score)
     for (int k = 0; k < top; ++k) {
-        float best = -1.f;
+        float best = -INFINITY;
         int at = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
             const float v = sc[e];
@@ -116,12 +124,20 @@ __global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, f
             ids[(size_t)t * top + k] = at;
             wts[(size_t)t * top + k] = best;
             rank[(size_t)t * top + k] = atomicAdd(&counts[at], 1);
-            sc[at] = -2.f;
+            sc[at] = -INFINITY;
         }
+        if (lane == k) mine = best;
+        if (k == 0) first = best;
         sum += best;
         __syncwarp();
     }
     __syncwarp();
+    if (score == MOE_LOGITS) {                           // softmax over the chosen logits, the first of which is the largest
+        const float w = lane < top ? expf(mine - first) : 0.f;
+        const float total = warp_sum(w);
+        if (lane < top) wts[(size_t)t * top + lane] = w / total;
+        return;
+    }
     if (renorm && lane < top) wts[(size_t)t * top + lane] /= sum + 1e-20f;
 }
 
@@ -182,7 +198,8 @@ template <> __device__ __forceinline__ void moe_store<float>(float* p, float v) 
 template <> __device__ __forceinline__ void moe_store<bf16>(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 __device__ __forceinline__ float moe_silu(float g) { return g / (1.f + expf(-g)); }
-// The gated epilogues: 1  silu(g) u;  2  g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+// The gated epilogues: 1  silu(g) u;  2  g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
+// Without a gate: 0  v;  3  relu(v)^2
 struct MoeAct {
     int kind;
     float limit, alpha;
@@ -191,6 +208,11 @@ struct MoeAct {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
         return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    }
+    __device__ __forceinline__ float plain(float v) const {
+        if (kind != 3) return v;
+        v = fmaxf(v, 0.f);
+        return v * v;
     }
 };
 
@@ -286,8 +308,8 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(TO* __restrict__ out,
         for (int c = 0; c < 2; ++c) {
             const int n = blockIdx.y * MOE_TN + (wn * NT + nt) * 8 + 2 * tq + c;
             if (n < n_out) {
-                moe_store<TO>(out + ra * n_out + n, acc[nt][c]);
-                moe_store<TO>(out + rb * n_out + n, acc[nt][2 + c]);
+                moe_store<TO>(out + ra * n_out + n, act.plain(acc[nt][c]));
+                moe_store<TO>(out + rb * n_out + n, act.plain(acc[nt][2 + c]));
             }
         }
     }
@@ -341,18 +363,20 @@ __global__ void __launch_bounds__(128) moe_gemm_plain_kernel(TO* __restrict__ ou
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
         const int n = blockIdx.y * MOE_TN + c8 + 8 * j;
-        if (n < n_out) moe_store<TO>(out + (row0 + r) * n_out + n, acc[j]);
+        if (n < n_out) moe_store<TO>(out + (row0 + r) * n_out + n, act.plain(acc[j]));
     }
 }
 
 // ------------------------------------------------------------------------------------------------ combine
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ y, const int* __restrict__ dest,
-                                   const float* __restrict__ wts, int W, int top, int scale_output) {
+                                   const float* __restrict__ wts, int W, int top, int scale_output, const T* __restrict__ unit,
+                                   const float* __restrict__ unit_gate) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
-    if ((W & 7) == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
+    const float ug = unit_gate ? unit_gate[t] : 1.f;     // (`unit`: the rows of the unit beside the experts)
+    if ((W & 7) == 0 && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(unit)) & 15) == 0) {
         for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {      // the same sums in the same order, eight columns at a time
             float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             for (int k = 0; k < top; ++k) {
@@ -361,6 +385,12 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
                 const float wk = scale_output ? wts[(size_t)t * top + k] : 1.f;
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[i] += scale_output ? v[i] * wk : v[i];
+            }
+            if (unit) {
+                float v[8];
+                moe_load8(v, unit + (size_t)t * W + c);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[i] += ug * v[i];
             }
             moe_store8(out + (size_t)t * W + c, acc);
         }
@@ -372,20 +402,24 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
             const float v = y[(size_t)dest[(size_t)t * top + k] * W + c];
             acc += scale_output ? v * wts[(size_t)t * top + k] : v;
         }
+        if (unit) acc += ug * to_float(unit[(size_t)t * W + c]);
         out[(size_t)t * W + c] = from_float<T>(acc);
     }
 }
 
 // ------------------------------------------------------------------------------------------------ launchers
-// ids, rank [N, top] int; wts [N, top] 32-bit; counts [E] int, zeroed here; x [N, x_stride] in `dtype`; wr [E, W] 32-bit
+// ids, rank [N, top] int; wts [N, top] 32-bit; counts [E] int, zeroed here; x [N, x_stride] in `dtype`; wr [E, W] 32-bit.
+// score: 0 sigmoid, 1 softmax over all experts, 2 the logits with softmax over the chosen (`bias` [E] 32-bit or null is added to
+// the logits; modes 1 and 2).  With `unit_gate` [N] wr has one row more, whose product's sigmoid goes there.
 ZAI_API int zai_moe_route(int* ids, float* wts, int* rank, int* counts, const void* x, int x_stride, int dtype, const float* wr,
-                          int N, int W, int E, int top, int renorm, int softmax, cudaStream_t stream) {
+                          int N, int W, int E, int top, int renorm, int score, const float* bias, float* unit_gate,
+                          cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
-    if (E < 1 || top < 1 || top > E || top > 32 || E > 8192 || W < 1) return ZAI_BAD_SIZE;
+    if (E < 1 || top < 1 || top > E || top > 32 || E > 8192 || W < 1 || score < MOE_SIGMOID || score > MOE_LOGITS || (bias && score == MOE_SIGMOID)) return ZAI_BAD_SIZE;
     cudaError_t rc = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int), stream);
     if (rc != cudaSuccess) return (int)rc;
     ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T>, dim3(N), dim3(128), (size_t)E * sizeof(float), stream, ids, wts, rank,
-                                          counts, (const T*)x, x_stride, wr, W, E, top, renorm, softmax));
+                                          counts, (const T*)x, x_stride, wr, W, E, top, renorm, score, bias, unit_gate));
 }
 
 // The most tiles of TM rows that N x top choices over E experts can take.
@@ -408,12 +442,14 @@ ZAI_API int zai_moe_gather(void* xs, int* dest, int* tile_expert, const void* x,
 }
 
 // out [max_tiles * TM, n_out] (32-bit if out_f32, else `dtype`) = xs [max_tiles * TM, K] . w[expert of the tile]^T;
-// w [E, n_out, K], or with `gated` [E, 2 n_out, K] and out = silu(gate) * up (gated 1) or the bounded gated activation with
-// `limit` and `alpha` (gated 2).  TM 16 or 64 (the gather's).
+// w [E, n_out, K], or with kind 1 or 2 [E, 2 n_out, K] and out = silu(gate) * up (kind 1) or the bounded gated activation with
+// `limit` and `alpha` (kind 2); kind 3: the square of relu on the plain products.  TM 16 or 64 (the gather's).
 ZAI_API int zai_moe_gemm(void* out, int out_f32, const void* xs, const void* w, int dtype, const int* tile_expert, int max_tiles,
-                         int TM, int K, int n_out, int gated, float limit, float alpha, cudaStream_t stream) {
+                         int TM, int K, int n_out, int kind, float limit, float alpha, cudaStream_t stream) {
     if (max_tiles <= 0) return ZAI_OK;
-    const MoeAct act = {gated, limit, alpha};
+    if (kind < 0 || kind > 3) return ZAI_BAD_SIZE;
+    const MoeAct act = {kind, limit, alpha};
+    const int gated = kind == 1 || kind == 2;
     if (K < 1 || n_out < 1 || (TM != 16 && TM != 64)) return ZAI_BAD_SIZE;
     const int cols = gated ? MOE_TN / 2 : MOE_TN;
     const dim3 grid(max_tiles, (n_out + cols - 1) / cols);
@@ -437,10 +473,11 @@ ZAI_API int zai_moe_gemm(void* out, int out_f32, const void* xs, const void* w, 
                       tile_expert, K, n_out, gated, act);
 }
 
-// out [N, W] in `dtype` = sum over a row's choices of y[dest], times the choice's weight with `scale_output`
+// out [N, W] in `dtype` = sum over a row's choices of y[dest], times the choice's weight with `scale_output`; plus, with `unit`
+// [N, W] in `dtype`, that row times unit_gate[row] (32-bit; null: times 1)
 ZAI_API int zai_moe_combine(void* out, int dtype, const float* y, const int* dest, const float* wts, int N, int W, int top,
-                            int scale_output, cudaStream_t stream) {
+                            int scale_output, const void* unit, const float* unit_gate, cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
     ZAI_DISPATCH(dtype, return launch_pdl(moe_combine_kernel<T>, dim3(N), dim3(W >= 1024 ? 256 : 128), 0, stream, (T*)out, y, dest,
-                                          wts, W, top, scale_output));
+                                          wts, W, top, scale_output, (const T*)unit, unit_gate));
 }

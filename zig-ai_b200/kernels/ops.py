@@ -28,6 +28,7 @@ _P, _I, _F = c_void_p, c_int, c_float
 _SIGNATURES = {
     "embed": {
         "zai_embed": [_P, _P, _I, _P, _I, _I, _I, _F, _P, _P],
+        "zai_embed_sinusoidal": [_P, _P, _I, _P, _I, _I, _I, _F, _P, _P, _P, _P],
         "zai_gather_add": [_P, _P, _P, _I, _P, _I, _I, _P],
         "zai_gather_add_normed": [_P, _P, _P, _I, _P, _F, _P, _I, _I, _P],
     },
@@ -35,11 +36,20 @@ _SIGNATURES = {
              "zai_add_normed_rmsnorm": [_P, _P, _P, _F, _P, _P, _I, _F, _I, _I, _P],
              "zai_add_normed_cast": [_P, _P, _P, _F, _P, _I, _I, _I, _P],
              "zai_rmsnorm_rows": [_P, _P, _I, _I, _P, _F, _I, _I, _P]},
-    "moe": {"zai_moe_route": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P],
+    "moe": {"zai_moe_route": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P],
             "zai_moe_max_tiles": [_I, _I, _I, _I],
             "zai_moe_gather": [_P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
             "zai_moe_gemm": [_P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _P],
-            "zai_moe_combine": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P]},
+            "zai_moe_combine": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P]},
+    "attention_difference": {"zai_attention_difference": [_P, _P, _I, _F, _F, _F, _I, _I, _I, _I, _P]},
+    "mamba2": {
+        "zai_mamba2_chunked_supports": [_I, _I],
+        "zai_mamba2_chunk_rows": [],
+        "zai_mamba2_scan": [_P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
+        "zai_mamba2_chunked": [_P, _P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P],
+        "zai_mamba2_single": [_P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
+        "zai_mamba2_norm": [_P, _P, _P, _I, _I, _I, _P, _F, _I, _I, _I, _P, _I, _I, _I, _P, _I, _P, _P],
+    },
     "layernorm": {"zai_add_layernorm": [_P, _P, _P, _P, _P, _I, _F, _I, _I, _P]},
     "qkv_prepare": {
         "zai_qkv_prepare": [_P, _I, _I, _P, _P, _F, _I, _P, _I, _P, _P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P,
@@ -101,6 +111,7 @@ _SIGNATURES = {
         "zai_skinny_gemm_supports": [_I, _I, _I, _I, _I],
         "zai_skinny_gemm": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _P],
         "zai_skinny_gemm_clamped_glu": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _F, _F, _P],
+        "zai_skinny_gemm_relu2": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _P],
         "zai_skinny_gemm_layernorm": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _F, _F, _P],
         "zai_skinny_conv": [_P, _P, _P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
         "zai_skinny_hint_next": [_P, ctypes.c_longlong],
@@ -360,14 +371,21 @@ fuses_layernorm = True  # ... also one that is a layer norm (`LazyNorm.beta`)
 
 _EPI_BF16, _EPI_F32, _EPI_SWIGLU = 0, 1, 2
 _EPI_F32_PAIR = 3          # (grouped tcgen05 products) 32-bit results, two weight tiles a stage
+_EPI_RELU2 = 4             # (grouped tcgen05 products) bfloat16, the square of relu
 
 
 @_timed("embedding")
-def embed(ids, table, scale=1.0):
-    """Rows of the table as 32-bit residual rows, times `scale`."""
-    _cuda(ids, table)
+def embed(ids, table, scale=1.0, positions=None, base=10000.0):
+    """Rows of the table as 32-bit residual rows, times `scale`; with `positions` [N] the sinusoidal vector of each row's
+    position is added: entries 2i and 2i + 1 are sine and cosine of position * base^(-2i/width)."""
+    _cuda(ids, table, positions)
     N, (V, H) = ids.numel(), table.shape
     out = torch.empty((N, H), dtype=torch.float32, device=table.device)
+    if positions is not None:
+        _check(_fn("embed", "zai_embed_sinusoidal")(_ptr(out), _ptr(table), _dt(table), _ptr(ids), N, H, V, float(scale), _ptr(positions),
+                                                    _ptr(sinusoidal_frequencies(H, base, table.device)), _status_ptr(table.device),
+                                                    _stream()), "embed_sinusoidal")
+        return out
     _check(_fn("embed", "zai_embed")(_ptr(out), _ptr(table), _dt(table), _ptr(ids), N, H, V, float(scale),
                                      _status_ptr(table.device), _stream()), "embed")
     return out
@@ -470,9 +488,9 @@ def _bias_through(w, beta):
 
 
 @_timed(_product_class)
-def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None):
+def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None):
     """The few-rows product kernel, if it takes these operands; else None.  `glu` = (limit, slope): the gated epilogue
-    with bounded branches instead of SiLU(gate) * up."""
+    with bounded branches instead of SiLU(gate) * up.  `plain_act="relu2"`: the square of relu as the bfloat16 epilogue."""
     lazy = isinstance(x, LazyNorm)
     M = (x.rows.numel() if x.rows is not None else x.residual.data.shape[0]) if lazy else x.shape[0]
     O, K = w.shape
@@ -482,9 +500,13 @@ def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None):
         return None
     if not _fn("decode_gemm", "zai_skinny_gemm_supports")(M, O, K, epilogue, int(lazy)):
         return None
+    if plain_act is not None and lazy and getattr(x, "beta", None) is not None:
+        return None
     y = torch.empty((M, out_cols), dtype=out_dtype, device=w.device)
     _hint_next_weights(w)
-    if glu is not None:
+    if plain_act is not None:
+        fn, tail = _fn("decode_gemm", "zai_skinny_gemm_relu2"), (_stream(),)
+    elif glu is not None:
         fn, tail = _fn("decode_gemm", "zai_skinny_gemm_clamped_glu"), (float(glu[0]), float(glu[1]), _stream())
     else:
         fn, tail = _fn("decode_gemm", "zai_skinny_gemm"), (epilogue, _stream())
@@ -779,6 +801,16 @@ def short_conv(bcx, conv_w, conv_b, state, step, taps, write_state=True):
 
 
 _inv_freq_cache = {}
+
+
+def sinusoidal_frequencies(width: int, base: float, device) -> torch.Tensor:
+    """base^(-2i/width) for every pair (2i, 2i + 1) of `width` entries, in 64-bit."""
+    key = ("sinusoidal", int(width), float(base), str(device))
+    t = _inv_freq_cache.get(key)
+    if t is None:
+        i = torch.arange((width + 1) // 2, dtype=torch.float64)
+        t = _inv_freq_cache[key] = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / width).to(device)
+    return t
 
 
 def inverse_frequencies(rotary_dim: int, theta: float, device, scaling=None) -> torch.Tensor:
@@ -1113,12 +1145,12 @@ def sample(logits, temperature, top_k, top_p, u, with_status=False):
 
 
 # ----------------------------------------------------------------------------- recurrent mixers and what goes with them
-ACTIVATIONS = {"gelu": 0, "gelu_erf": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
+ACTIVATIONS = {"gelu": 0, "gelu_erf": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "relu2": 4}
 
 
 @_timed("activation")
 def activation(x, kind):
-    """An activation by name (gelu / gelu_erf, gelu_tanh, silu, relu), computed in 32-bit."""
+    """An activation by name (gelu / gelu_erf, gelu_tanh, silu, relu, relu2: relu squared), computed in 32-bit."""
     _cuda(x)
     out = torch.empty_like(x)
     _check(_fn("activation", "zai_activation")(_ptr(out), _ptr(x), _dt(x), ACTIVATIONS[kind], x.numel(), _stream()), "activation")
@@ -1126,7 +1158,12 @@ def activation(x, kind):
 
 
 def linear_activation(x, w, kind):
-    """act(x . w^T): the product (x may be a LazyNorm), then the activation."""
+    """act(x . w^T): the product (x may be a LazyNorm), then the activation (relu squared: the product's epilogue for few rows
+    in bfloat16)."""
+    if kind == "relu2" and x.dtype == torch.bfloat16:
+        y = _skinny(x, w, _EPI_BF16, w.shape[0], torch.bfloat16, plain_act="relu2")
+        if y is not None:
+            return y
     return activation(linear(x, w), kind)
 
 
@@ -1495,23 +1532,31 @@ MOE_TALL_TILE_ROWS = 32      # from this many rows per expert on average, tiles 
 
 @_timed("experts")
 def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on="input", score="sigmoid", act="silu", limit=0.0,
-                   alpha=1.702):
+                   alpha=1.702, router_bias=None, unit=None, unit_gated=False):
     """A mixture of gated feed-forwards.  x [N, W]; w_router [E, W] 32-bit; w_gate_up [E, 2 F, W] (an expert's gate rows,
     then its up rows); w_down [E, W, F].  Every row goes to the `top` experts with the largest sigmoid(x . w_router^T)
     (32-bit); the scores are the weights (divided by their sum with `renorm`), applied to the expert's input or to its
     output; the row's results are summed in 32-bit.  Nothing is read back to the host.  `score="softmax"`: the scores are the
     softmax of the router's logits over all experts (`renorm` divides by the chosen scores' sum + 1e-20).  `act="clamped"`:
-    the experts are bounded gated units min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1)."""
-    if score not in ("sigmoid", "softmax") or act not in ("silu", "clamped"):
-        raise KernelError("routed_experts: score is sigmoid or softmax, act silu or clamped")
-    gated = 2 if act == "clamped" else 1
-    _cuda(w_router, w_gate_up, w_down)
+    the experts are bounded gated units min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1).
+    `score="chosen"`: the logits themselves choose and the weights are the softmax over the chosen logits.  `router_bias` [E]
+    32-bit is added to the logits (not with sigmoid scores).  `act="relu2"`: experts without a gate, down(relu(up)^2), w_gate_up
+    being [E, F, W].  `unit` [N, W]: the rows of a feed-forward that every row passes, added in the same sum; with `unit_gated`
+    times sigmoid(x . w), w being the row of w_router [E + 1, W] behind the experts'."""
+    if score not in ("sigmoid", "softmax", "chosen") or act not in ("silu", "clamped", "relu2"):
+        raise KernelError("routed_experts: score is sigmoid, softmax or chosen, act silu, clamped or relu2")
+    gated = {"silu": 1, "clamped": 2, "relu2": 3}[act]
+    _cuda(w_router, w_gate_up, w_down, router_bias, unit)
     xp, xs = _rows_view(x)
     N, W = x.shape
-    E, F = w_gate_up.shape[0], w_gate_up.shape[1] // 2
+    E, up_rows = w_gate_up.shape[0], w_gate_up.shape[1]
+    F = up_rows if act == "relu2" else up_rows // 2
     top = int(top)
-    if (w_router.dtype != torch.float32 or tuple(w_router.shape) != (E, W) or tuple(w_gate_up.shape) != (E, 2 * F, W)
-            or tuple(w_down.shape) != (E, W, F) or w_gate_up.dtype != x.dtype or w_down.dtype != x.dtype
+    if unit_gated and unit is None or (unit is not None and (tuple(unit.shape) != (N, W) or unit.dtype != x.dtype)) or (
+            router_bias is not None and (router_bias.dtype != torch.float32 or router_bias.numel() != E or score == "sigmoid")):
+        raise KernelError("routed_experts: the router's bias or the unit's rows do not fit")
+    if (w_router.dtype != torch.float32 or tuple(w_router.shape) != (E + int(unit_gated), W) or up_rows != (F if act == "relu2" else 2 * F)
+            or w_gate_up.shape[2] != W or tuple(w_down.shape) != (E, W, F) or w_gate_up.dtype != x.dtype or w_down.dtype != x.dtype
             or weight_on not in ("input", "output")):
         raise KernelError("routed_experts: operands do not fit together")
     dev, dt, lib = x.device, _dt(x), "moe"
@@ -1521,19 +1566,21 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
     tall = dt == _BF16 and W % 8 == 0 and F % 8 == 0 and N * top >= MOE_TALL_TILE_ROWS * E
     # many rows an expert: tiles of 128 rows and both products on the 5th-generation tensor cores (grouped tcgen05)
     grouped = (tall and USE_MOE_GROUPED_TC and N * top >= MOE_GROUPED_TILE_ROWS * E
-               and _fn("gemm_tc", "zai_gemm_tc_supports")(128, 2 * F, W, _EPI_SWIGLU if act == "silu" else _EPI_BF16)
+               and _fn("gemm_tc", "zai_gemm_tc_supports")(128, up_rows, W, _EPI_SWIGLU if act == "silu" else _EPI_BF16)
                and _fn("gemm_tc", "zai_gemm_tc_supports")(128, W, F, _EPI_F32))
     TM = 128 if grouped else 64 if tall else 16
     max_tiles = _fn(lib, "zai_moe_max_tiles")(N, top, E, TM)
     if max_tiles < 0:
         raise KernelError("routed_experts: too many rows")
-    meta = torch.empty((4 * N * top + E + max_tiles,), dtype=torch.int32, device=dev)
+    meta = torch.empty((4 * N * top + E + max_tiles + N,), dtype=torch.int32, device=dev)
     ids, rank, dest = meta[:N * top], meta[N * top:2 * N * top], meta[2 * N * top:3 * N * top]
     wts = meta[3 * N * top:4 * N * top].view(torch.float32)
-    counts, tile_expert = meta[4 * N * top:4 * N * top + E], meta[4 * N * top + E:]
+    counts, tile_expert = meta[4 * N * top:4 * N * top + E], meta[4 * N * top + E:4 * N * top + E + max_tiles]
+    unit_gate = meta[4 * N * top + E + max_tiles:].view(torch.float32) if unit_gated else None
     on_input = int(weight_on == "input")
     _check(_fn(lib, "zai_moe_route")(_ptr(ids), _ptr(wts), _ptr(rank), _ptr(counts), xp, xs, dt, _ptr(w_router), N, W, E, top,
-                                     int(bool(renorm)), int(score == "softmax"), _stream()), "moe_route")
+                                     int(bool(renorm)), {"sigmoid": 0, "softmax": 1, "chosen": 2}[score], _ptr(router_bias),
+                                     _ptr(unit_gate), _stream()), "moe_route")
     rows = max_tiles * TM
     x_sorted = torch.empty((rows, W), dtype=x.dtype, device=dev)
     _check(_fn(lib, "zai_moe_gather")(_ptr(x_sorted), _ptr(dest), _ptr(tile_expert), xp, xs, dt, _ptr(ids), _ptr(wts), _ptr(rank),
@@ -1548,19 +1595,21 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
                       _EPI_BF16, _stream()), "gemm_tc_grouped (gate/up)")
             hidden = clamped_glu(gu, F, limit, alpha)
         else:
-            _check(tc(_ptr(hidden), _ptr(w_gate_up), _ptr(x_sorted), _ptr(tile_expert), _status_ptr(dev), max_tiles, E, 2 * F, W,
-                      _EPI_SWIGLU, _stream()), "gemm_tc_grouped (gate/up)")
+            _check(tc(_ptr(hidden), _ptr(w_gate_up), _ptr(x_sorted), _ptr(tile_expert), _status_ptr(dev), max_tiles, E, up_rows, W,
+                      _EPI_RELU2 if act == "relu2" else _EPI_SWIGLU, _stream()), "gemm_tc_grouped (gate/up)")
         _check(tc(_ptr(y), _ptr(w_down), _ptr(hidden), _ptr(tile_expert), _status_ptr(dev), max_tiles, E, W, F,
                   _EPI_F32_PAIR if USE_MOE_DOWN_PAIR else _EPI_F32, _stream()),
                "gemm_tc_grouped (down)")
-        _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _stream()),
+        _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _ptr(unit),
+                                               _ptr(unit_gate), _stream()),
                "moe_combine")
         return out
     _check(_fn(lib, "zai_moe_gemm")(_ptr(hidden), int(dt == _F32), _ptr(x_sorted), _ptr(w_gate_up), dt, _ptr(tile_expert), max_tiles,
                                     TM, W, F, gated, float(limit), float(alpha), _stream()), "moe_gemm (gate/up)")
     _check(_fn(lib, "zai_moe_gemm")(_ptr(y), 1, _ptr(hidden), _ptr(w_down), dt, _ptr(tile_expert), max_tiles, TM, F, W, 0, 0.0, 0.0,
                                     _stream()), "moe_gemm (down)")
-    _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _stream()),
+    _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _ptr(unit),
+                                               _ptr(unit_gate), _stream()),
            "moe_combine")
     return out
 
@@ -1590,6 +1639,75 @@ def linear_glu(x, w_gate_up, ff_dim, kind):
         if y is not None:
             return y
     return act_mul(linear(x, w_gate_up), ff_dim, kind)
+
+
+@_timed("attention")
+def attention_difference(o, heads, vdim, cache_dim, lam, factor, eps):
+    """The two maps of differential attention combined: o [N, 2 * heads * cache_dim] with a head's maps side by side;
+    factor * d / rms(d) per head, d = o1 - lam * o2 over the head's `vdim` values, [N, heads * vdim]."""
+    _cuda(o)
+    N, H, Dv, Dp = o.shape[0], int(heads), int(vdim), int(cache_dim)
+    if o.shape[1] != 2 * H * Dp:
+        raise KernelError("attention_difference: the rows do not hold two maps of every head")
+    out = torch.empty((N, H * Dv), dtype=o.dtype, device=o.device)
+    _check(_fn("attention_difference", "zai_attention_difference")(_ptr(out), _ptr(o), _dt(o), float(lam), float(factor), float(eps), N, H,
+                                                                   Dv, Dp, _stream()), "attention_difference")
+    return out
+
+
+MAMBA2_CHUNKED_MIN = 24          # spans of this many rows or more run in chunks on the tensor cores (bfloat16)
+USE_MAMBA2_CHUNKS = os.environ.get("ZAI_MAMBA2_CHUNKS", "1") == "1"
+
+
+@_timed("recurrence")
+def mamba2(y, at, conv_w, conv_b, dt_bias, a_log, d_skip, norm_w, eps, norm_parts, state, conv_state, step, heads, groups, state_dim,
+           vdim, write_state=True, impl=None):
+    """The state-space recurrence with one decay per head.  y [N, cols]: the in-projection's rows, `at` the first columns of z (H
+    V), x | B | C (H V + 2 G Ns) and dt (H); conv_w [channels, L] and conv_b [channels] or None, dt_bias, a_log, d_skip [H],
+    norm_w [H V] 32-bit; state [slots, H, Ns, V] and conv_state [slots, L - 1, channels] 32-bit.  Returns the gated and normed
+    read-out, [N, H V] in y's dtype.  `impl` "walk" or "chunks" picks the kernels for spans whatever their length."""
+    _cuda(conv_w, conv_b, dt_bias, a_log, d_skip, norm_w, state, conv_state)
+    yp, ys = _rows_view(y)
+    N, H, G, Ns, V = y.shape[0], int(heads), int(groups), int(state_dim), int(vdim)
+    I, ch, L, lib, dev = H * V, H * V + 2 * G * Ns, conv_w.shape[1], "mamba2", y.device
+    z_at, xbc_at, dt_at = (int(a) for a in at)
+    if (state.dtype != torch.float32 or tuple(state.shape[1:]) != (H, Ns, V) or conv_state.dtype != torch.float32
+            or conv_w.shape[0] != ch or conv_state.shape[-1] != ch or (L > 1 and conv_state.shape[1] != L - 1) or N != step.n_tokens
+            or norm_w.numel() != I or any(t.dtype != torch.float32 or t.numel() != H for t in (dt_bias, a_log, d_skip))):
+        raise KernelError("mamba2: operands do not fit together")
+    o = torch.empty((N, I), dtype=torch.float32, device=dev)
+    out = torch.empty((N, I), dtype=y.dtype, device=dev)
+    status, wr = _status_ptr(dev), int(bool(write_state))
+    if step.decode_only and N == step.n_seqs and impl is None:
+        _check(_fn(lib, "zai_mamba2_single")(
+            _ptr(o), yp, ys, _dt(y), xbc_at, dt_at, _ptr(conv_w), _ptr(conv_b), _ptr(conv_state), L, _ptr(dt_bias), _ptr(a_log),
+            _ptr(d_skip), _ptr(state), _ptr(step.slot_ids), state.shape[0], status, N, H, G, Ns, V, wr, _stream()), "mamba2_single")
+        _check(_fn(lib, "zai_mamba2_norm")(_ptr(out), _ptr(o), yp, ys, _dt(y), z_at, _ptr(norm_w), float(eps), N, I, int(norm_parts),
+                                           _ptr(conv_state) if wr else None, xbc_at, ch, L, _ptr(step.slot_ids), state.shape[0], status,
+                                           _stream()), "mamba2_norm")
+        return out
+    u = causal_conv(y[:, xbc_at:xbc_at + ch], conv_w, conv_b, conv_state, step, True, write_state)
+    dtp = yp + dt_at * y.element_size()
+    # spans shorter than `cut` are walked row by row, the others run in chunks (spans of a step are of both kinds; which kernel a
+    # span takes depends on its own length alone)
+    cut = 1 << 30
+    if impl != "walk" and y.dtype == torch.bfloat16 and _fn(lib, "zai_mamba2_chunked_supports")(Ns, V) and (USE_MAMBA2_CHUNKS or impl == "chunks"):
+        cut = 1 if impl == "chunks" else MAMBA2_CHUNKED_MIN
+    if N >= cut:
+        rows = _fn(lib, "zai_mamba2_chunk_rows")()
+        max_chunks = N // rows + step.n_seqs
+        ends = torch.empty((max_chunks, H, Ns, V), dtype=torch.float32, device=dev)
+        last = torch.empty((max_chunks, H), dtype=torch.float32, device=dev)
+        _check(_fn(lib, "zai_mamba2_chunked")(
+            _ptr(o), _ptr(u), ch, dtp, ys, _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(state), _ptr(step.cu_q), _ptr(step.slot_ids),
+            state.shape[0], status, step.n_seqs, H, G, Ns, V, wr, cut, _ptr(ends), _ptr(last), max_chunks, _stream()), "mamba2_chunked", 3)
+    if cut > 1 and not (N >= cut and step.n_seqs == 1):
+        _check(_fn(lib, "zai_mamba2_scan")(
+            _ptr(o), _ptr(u), ch, dtp, ys, _dt(y), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(state), _ptr(step.cu_q),
+            _ptr(step.slot_ids), state.shape[0], status, step.n_seqs, H, G, Ns, V, wr, 1, cut - 1, _stream()), "mamba2_scan")
+    _check(_fn(lib, "zai_mamba2_norm")(_ptr(out), _ptr(o), yp, ys, _dt(y), z_at, _ptr(norm_w), float(eps), N, I, int(norm_parts), None, 0, 0,
+                                       1, None, 0, status, _stream()), "mamba2_norm")
+    return out
 
 
 @_timed("recurrence")

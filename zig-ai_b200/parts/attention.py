@@ -37,6 +37,16 @@ Options that shape the scores or the values (they also take the one-product path
                            caches (1 - lambda) v + lambda v_first with its learned scalar `vmix` (the first layer's is stored
                            and unused)
 
+`differential={"diff": c}`: differential attention.  The q and k projections hold two maps per head, side by side (q: heads x
+[map 1 | map 2] of D each, k the same per key/value head); each map is an attention of its own over the same values, and
+
+    lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + c      (four learned vectors of D, one lambda for the layer)
+    d = o1 - lambda o2;   o = (1 - c) d / sqrt(mean(d^2) + eps) per head over Dv      (no weight), then Wo
+
+A page keeps a key head's two maps as one key of 2 D values, and a head's maps run as two query heads [q1 | 0] and [0 | q2]
+of the same key/value head: the zeros change no score, keys and values are cached and read once, and every attention
+kernel serves as it is.  One kernel combines the two outputs (`ops.attention_difference`).
+
 Reference: projections src/transformer/hybrid_attn.zig:285-354, per-head norm :371-382 (device
 :719,723), scale 1/sqrt(D) :571, causal mask :587, softmax :578-600, query head hq reads kv head
 hq // (Hq/Hkv) :553-569 and src/cuda/paged_attention.cu:142, output projection :622-640; tensor
@@ -59,7 +69,15 @@ class Attention(Mixer):
     def __init__(self, hidden: int, heads: int, kv_heads: int, head_dim: int, qk_norm: bool, eps: float,
                  position: PartSpec, window=None, scale=None, kv_proj: bool = True, value_dim=None,
                  value_norm: bool = False, names=None, bias: bool = False, norm_scope: str = "head", chunk=None, gate=None,
-                 q_temp=None, softcap=None, rel_bias=None, sink: bool = False, keep_first: int = 0, v_mix=None):
+                 q_temp=None, softcap=None, rel_bias=None, sink: bool = False, keep_first: int = 0, v_mix=None, differential=None):
+        self.differential = None if differential is None else float(differential["diff"])
+        if self.differential is not None:
+            # to everything below, a head is a pair of query heads over keys of twice the size
+            plain = not (qk_norm or value_norm or bias or gate or chunk or q_temp or softcap or rel_bias or sink or keep_first or v_mix)
+            if not plain or not kv_proj or position.kind != "none" or scale is None or value_dim is None:
+                raise ValueError("differential attention goes with a window at most, and takes scale and value_dim")
+            self.map_heads, self.map_dim = int(heads), int(head_dim)
+            heads, head_dim = 2 * int(heads), 2 * int(head_dim)
         self.hidden, self.heads, self.kv_heads, self.head_dim = int(hidden), int(heads), int(kv_heads), int(head_dim)
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads cannot share {self.kv_heads} key/value heads evenly")
@@ -76,7 +94,8 @@ class Attention(Mixer):
         self.names = {"q": "attn_q.weight", "k": "attn_k.weight", "v": "attn_v.weight", "o": "attn_output.weight",
                       "q_norm": "attn_q_norm.weight", "k_norm": "attn_k_norm.weight", "q_bias": "attn_q.bias",
                       "k_bias": "attn_k.bias", "v_bias": "attn_v.bias", "g": "attn_gate.weight", "rel": "attn_rel_bias",
-                      "sink": "attn_sink", "vmix": "attn_vmix", **(names or {})}
+                      "sink": "attn_sink", "vmix": "attn_vmix", "lq1": "attn_lambda_q1", "lk1": "attn_lambda_k1",
+                      "lq2": "attn_lambda_q2", "lk2": "attn_lambda_k2", **(names or {})}
         self.bias, self.norm_scope, self.gate = bool(bias), str(norm_scope), gate
         self.chunk = None if chunk is None else int(chunk)
         if self.norm_scope not in ("head", "whole") or self.gate not in (None, "head"):
@@ -105,12 +124,19 @@ class Attention(Mixer):
             raise ValueError("value_norm and a borrowed cache are not combined with bias, whole norm, chunk or gate")
         if self.prepared:
             self.kernel_libs = type(self).kernel_libs + ("qkv_prepare",)
+        if self.differential is not None:
+            self.kernel_libs = type(self).kernel_libs + ("attention_difference",)
 
     def params(self):
         q_dim, kv_dim = self.heads * self.head_dim, self.kv_heads * self.head_dim
         nm = self.names
         p = {nm["q"]: ParamDecl((q_dim, self.hidden)),
              nm["o"]: ParamDecl((self.hidden, self.heads * self.value_dim))}
+        if self.differential is not None:
+            p = {nm["q"]: ParamDecl((self.map_heads * 2 * self.map_dim, self.hidden)),
+                 nm["o"]: ParamDecl((self.hidden, self.map_heads * self.value_dim))}
+            for k in ("lq1", "lk1", "lq2", "lk2"):
+                p[nm[k]] = ParamDecl((self.map_dim,), "vector", init="conv")
         if self.kv_proj:
             p[nm["k"]] = ParamDecl((kv_dim, self.hidden))
             p[nm["v"]] = ParamDecl((self.kv_heads * self.value_dim, self.hidden))
@@ -219,6 +245,10 @@ class Attention(Mixer):
             return self._bind_prepared(tensors, dtype)
         nm = self.names
         mats = [tensors[nm["q"]]]
+        if self.differential is not None:
+            mats = [self._two_maps(tensors[nm["q"]])]
+            vec = {k: tensors[nm[k]].double() for k in ("lq1", "lk1", "lq2", "lk2")}
+            self.lam = float(torch.exp((vec["lq1"] * vec["lk1"]).sum()) - torch.exp((vec["lq2"] * vec["lk2"]).sum())) + self.differential
         if self.kv_proj:
             mats += [tensors[nm["k"]], tensors[nm["v"]]]
         self.w_qkv = torch.cat(mats, dim=0).contiguous()
@@ -232,12 +262,26 @@ class Attention(Mixer):
             # mean_D = mean_Dp * Dp / D, so  rsqrt(mean_D + eps) = rsqrt(mean_Dp + eps D / Dp) * sqrt(D / Dp)
             grow = lambda g: None if g is None else torch.cat([g * (D / Dp) ** 0.5, g.new_zeros(Dp - D)]).contiguous()
             self.q_norm, self.k_norm, self.norm_eps = grow(self.q_norm), grow(self.k_norm), self.eps * D / Dp
-        if Dp != Dv:
+        if Dp != Dv and self.differential is None:
             # the heads come out of attention Dp wide with zeros behind their Dv values: the output
             # projection gets zero columns there
             w = self.w_o.reshape(self.hidden, self.heads, Dv)
             self.w_o = torch.cat([w, w.new_zeros(self.hidden, self.heads, Dp - Dv)], dim=2).reshape(self.hidden, -1).contiguous()
         self.dtype = dtype
+
+    def _two_maps(self, q):
+        """The rows of a q projection [H, map 1 | map 2] as 2 H heads of 2 D rows: [map 1 | 0], [0 | map 2]."""
+        H, D = self.map_heads, self.map_dim
+        w = q.reshape(H, 2, D, self.hidden)
+        out = w.new_zeros((H, 2, 2, D, self.hidden))
+        out[:, 0, 0], out[:, 1, 1] = w[:, 0], w[:, 1]
+        return out.reshape(4 * H * D, self.hidden)
+
+    def _output(self, o, ops):
+        """From the heads' outputs [N, heads * cache_dim] through the output projection."""
+        if self.differential is not None:
+            o = ops.attention_difference(o, self.map_heads, self.value_dim, self.cache_dim, self.lam, 1.0 - self.differential, self.eps)
+        return ops.linear(o, self.w_o)
 
     def forward(self, x, step, cache, write_cache=True):
         if self.prepared:
@@ -255,7 +299,7 @@ class Attention(Mixer):
             # the key chunks run as one kernel
             o = ops.decode_attention_fused(qkv, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache,
                                            self.heads, self.kv_heads, self.cache_dim, self.scale, self.window, write)
-            return ops.linear(o, self.w_o)
+            return self._output(o, ops)
         if rot is not None:
             q, _ = ops.qk_norm_rope(qkv, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache,
                                     self.heads, self.kv_heads, self.cache_dim, self.kv_proj, write, False)
@@ -267,7 +311,7 @@ class Attention(Mixer):
                 v = qkv[:, (self.heads + self.kv_heads) * self.cache_dim:]
                 ops.kv_write(k, v, step, cache, self.kv_heads, self.cache_dim)
         o = ops.paged_attention(q, step, cache, self.heads, self.kv_heads, self.cache_dim, self.scale, self.window)
-        return ops.linear(o, self.w_o)
+        return self._output(o, ops)
 
 
 register_part("mixer", "attention", Attention)

@@ -15,9 +15,14 @@ from .base import Embedding, Head, ParamDecl, register_part
 class TokenEmbedding(Embedding):
     graph_safe = True      # forward launches kernels only; nothing is read back to the host
 
-    def __init__(self, weight: str, vocab: int, hidden: int, scale: float = 1.0):
+    def __init__(self, weight: str, vocab: int, hidden: int, scale: float = 1.0, sinusoidal=None):
+        """`sinusoidal=base`: a vector of the token's position is added to its row, sines in the even and cosines in the odd
+        entries, entries 2i and 2i + 1 turning by base^(-2i/hidden) a position."""
         self.weight_name, self.vocab, self.hidden = weight, int(vocab), int(hidden)
         self.scale = float(scale)          # the gathered rows are multiplied by it (in 32-bit)
+        self.sinusoidal = None if sinusoidal is None else float(sinusoidal)
+        if self.sinusoidal is not None and self.sinusoidal <= 0:
+            raise ValueError("the base of the position vectors is positive")
         self.table = None
 
     def params(self):
@@ -27,6 +32,8 @@ class TokenEmbedding(Embedding):
         self.table = tensors[self.weight_name]
 
     def forward(self, token_ids, step):
+        if self.sinusoidal is not None:
+            return step.ops.embed(token_ids, self.table, self.scale, step.positions, self.sinusoidal)
         if self.scale != 1.0:
             return step.ops.embed(token_ids, self.table, self.scale)
         return step.ops.embed(token_ids, self.table)

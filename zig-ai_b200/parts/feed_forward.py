@@ -48,13 +48,13 @@ class SwiGlu(FeedForward):
 
 class DenseMlp(FeedForward):
     """`down( act(up(x)) )`, no gate and no biases; `activation` is one of gelu (the exact one, with erf),
-    gelu_tanh, silu, relu.  `names` gives the two tensors' names."""
+    gelu_tanh, silu, relu, relu2 (the square of relu).  `names` gives the two tensors' names."""
     accepts_lazy_input = True     # x goes straight into a product
     graph_safe = True
 
     def __init__(self, hidden: int, ff_dim: int, activation: str = "gelu", names=None):
         self.hidden, self.ff_dim, self.activation = int(hidden), int(ff_dim), str(activation)
-        if self.activation not in ("gelu", "gelu_erf", "gelu_tanh", "silu", "relu"):
+        if self.activation not in ("gelu", "gelu_erf", "gelu_tanh", "silu", "relu", "relu2"):
             raise ValueError(f"unknown activation '{self.activation}'")
         self.names = {"up": "ffn_up.weight", "down": "ffn_down.weight", **(names or {})}
 
@@ -114,32 +114,48 @@ class RoutedExperts(FeedForward):
     Options: `score="softmax"` (s = softmax of the router's logits over all experts; with `renormalize` the chosen scores
     are divided by their sum + 1e-20); `expert_act="clamped"` with `limit` and `alpha` (experts of the bounded form
     min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + 1)); `shared`, the `PartSpec` of a feed-forward
-    that every token passes beside its experts (its tensors under its own names) and whose output is added."""
+    that every token passes beside its experts (its tensors under its own names) and whose output is added.
+
+    `score="chosen"`: the logits choose and the weights are the softmax over the chosen logits alone; `router_bias` adds a
+    learned number per expert (name "router_bias") to the logits.  `expert_act="relu2"`: experts without a gate,
+    down_e( relu(up_e(x))^2 ).  `shared_gate`: the shared feed-forward's output times sigmoid(x . w) with a learned row w (name
+    "shared_gate"), computed in 32-bit with the router."""
     accepts_lazy_input = False    # the router and the experts read the normed rows themselves
     graph_safe = True             # routing stays on the device: forward launches kernels only
     kernel_libs = ("moe", "gemm_tc")      # (gemm_tc: the grouped products of steps with many rows an expert, bfloat16)
 
     def __init__(self, hidden: int, ff_dim: int, experts: int, top: int, renormalize: bool = False, weight_on: str = "input",
-                 names=None, score: str = "sigmoid", expert_act: str = "silu", limit: float = 0.0, alpha: float = 1.702, shared=None):
+                 names=None, score: str = "sigmoid", expert_act: str = "silu", limit: float = 0.0, alpha: float = 1.702, shared=None,
+                 router_bias: bool = False, shared_gate: bool = False):
         self.hidden, self.ff_dim, self.experts, self.top = int(hidden), int(ff_dim), int(experts), int(top)
         self.renormalize, self.weight_on = bool(renormalize), weight_on
         if not 1 <= self.top <= self.experts or self.top > 32:
             raise ValueError(f"a token uses between 1 and min(experts, 32) experts, not {self.top} of {self.experts}")
         if weight_on not in ("input", "output"):
             raise ValueError("weight_on is 'input' or 'output'")
-        if score not in ("sigmoid", "softmax") or expert_act not in ("silu", "clamped"):
-            raise ValueError("score is 'sigmoid' or 'softmax', expert_act 'silu' or 'clamped'")
+        if score not in ("sigmoid", "softmax", "chosen") or expert_act not in ("silu", "clamped", "relu2"):
+            raise ValueError("score is 'sigmoid', 'softmax' or 'chosen', expert_act 'silu', 'clamped' or 'relu2'")
+        self.router_bias, self.shared_gate = bool(router_bias), bool(shared_gate)
+        if self.router_bias and score == "sigmoid":
+            raise ValueError("a router bias goes with softmax or chosen-logit scores")
+        if self.shared_gate and shared is None:
+            raise ValueError("a gate on the shared feed-forward needs one")
         self.score, self.expert_act, self.limit, self.alpha = score, expert_act, float(limit), float(alpha)
         self.shared = None if shared is None else make_part("feed_forward", shared)
         if self.shared is not None:
             self.kernel_libs = type(self).kernel_libs + tuple(getattr(self.shared, "kernel_libs", ()))
-        self.names = {"router": "ffn_router.weight", "gate": "ffn_gate.{e}.weight", "up": "ffn_up.{e}.weight",
+        self.names = {"router": "ffn_router.weight", "router_bias": "ffn_router.bias", "shared_gate": "ffn_shared_gate.weight", "gate": "ffn_gate.{e}.weight", "up": "ffn_up.{e}.weight",
                       "down": "ffn_down.{e}.weight", **(names or {})}
 
     def params(self):
         nm, p = self.names, {self.names["router"]: ParamDecl((self.experts, self.hidden), "vector", init="conv")}
+        if self.router_bias:
+            p[nm["router_bias"]] = ParamDecl((self.experts,), "vector", init="conv")
+        if self.shared_gate:
+            p[nm["shared_gate"]] = ParamDecl((1, self.hidden), "vector", init="conv")
         for e in range(self.experts):
-            p[nm["gate"].format(e=e)] = ParamDecl((self.ff_dim, self.hidden))
+            if self.expert_act != "relu2":
+                p[nm["gate"].format(e=e)] = ParamDecl((self.ff_dim, self.hidden))
             p[nm["up"].format(e=e)] = ParamDecl((self.ff_dim, self.hidden))
             p[nm["down"].format(e=e)] = ParamDecl((self.hidden, self.ff_dim))
         if self.shared is not None:
@@ -150,14 +166,27 @@ class RoutedExperts(FeedForward):
         nm, E = self.names, range(self.experts)
         if self.shared is not None:
             self.shared.bind({k: tensors[k] for k in self.shared.params()}, dtype)
-        self.w_router = tensors[nm["router"]].float().contiguous()
-        self.w_gate_up = torch.stack([torch.cat([tensors[nm["gate"].format(e=e)], tensors[nm["up"].format(e=e)]], dim=0)
-                                      for e in E]).contiguous()                                  # [E, 2F, hidden]
+        self.w_router = tensors[nm["router"]].float()
+        if self.shared_gate:                 # one more row of the router's product
+            self.w_router = torch.cat([self.w_router, tensors[nm["shared_gate"]].float().reshape(1, self.hidden)], dim=0)
+        self.w_router = self.w_router.contiguous()
+        self.b_router = tensors[nm["router_bias"]].float().contiguous() if self.router_bias else None
+        if self.expert_act == "relu2":
+            self.w_gate_up = torch.stack([tensors[nm["up"].format(e=e)] for e in E]).contiguous()  # [E, F, hidden]
+        else:
+            self.w_gate_up = torch.stack([torch.cat([tensors[nm["gate"].format(e=e)], tensors[nm["up"].format(e=e)]], dim=0)
+                                          for e in E]).contiguous()                              # [E, 2F, hidden]
         self.w_down = torch.stack([tensors[nm["down"].format(e=e)] for e in E]).contiguous()   # [E, hidden, F]
         self.dtype = dtype
 
     def forward(self, x, step):
         ops = step.ops
+        if self.score == "chosen" or self.expert_act == "relu2" or self.router_bias or self.shared_gate:
+            # the shared feed-forward's rows join in the sum over the chosen experts
+            unit = None if self.shared is None else self.shared.forward(x, step)
+            return ops.routed_experts(x, self.w_router, self.w_gate_up, self.w_down, self.top, self.renormalize, self.weight_on,
+                                      score=self.score, act=self.expert_act, limit=self.limit, alpha=self.alpha,
+                                      router_bias=self.b_router, unit=unit, unit_gated=self.shared_gate)
         if self.score == "sigmoid" and self.expert_act == "silu":
             y = ops.routed_experts(x, self.w_router, self.w_gate_up, self.w_down, self.top, self.renormalize, self.weight_on)
         else:
