@@ -252,6 +252,8 @@ def run_ours(args):
         return run_zikevik(args)
     if args.only == "lolivik":
         return run_lolivik(args)
+    if args.only == "sogenex":
+        return run_sogenex(args)
     if args.only == "long":
         return run_long(args)
     if args.only == "sample":
@@ -381,7 +383,8 @@ def engine_numbers(eng):
     for blk in eng.runner.model.blocks:
         ff = getattr(blk, "feed_forward", None)
         if ff is not None and hasattr(ff, "experts") and hasattr(ff, "top"):
-            routed.append((ff.experts, ff.top, 3 * ff.hidden * ff.ff_dim))
+            per = 2 if getattr(ff, "expert_act", "") == "relu2" else 3            # matrices an expert has
+            routed.append((ff.experts, ff.top, per * ff.hidden * ff.ff_dim))
     return dict(matrix_params=matrix, kv_bytes_per_token=cache.bytes_per_token(), state_bytes=state, routed=routed)
 
 
@@ -800,19 +803,18 @@ def zikevik_kernel_rooflines(width, hbm_peak, flops_peak):
              "GB_per_s": round(by / ms / 1e6, 1), "of_copy_peak": round(by / ms / 1e6 / hbm_peak, 4)} for k, p, ms, fl, by in rows]
 
 
-def run_zikevik(args):
-    """Prefill and decode throughput of the Zikevik design at two widths beside the Pikasun design (the closest one:
-    latent attention in front of gated feed-forwards) of the same width, layer count and vocabulary; the time of a prefill
-    and of a decode step by kernel class; and its kernels alone beside the like kernels.  JSON lines, then markdown."""
+def run_beside(args, models_at, kernel_rooflines):
+    """Prefill and decode throughput of the models `models_at(width)` (label, config) at two widths, the time of a prefill and
+    of a decode step by kernel class, and the kernels of `kernel_rooflines(width, ...)` alone.  JSON lines, then markdown."""
     import torch
     import zig_ai_b200 as z
     from zig_ai_b200.config import config_from_dict
     hbm_peak, flops_peak, peak_src = peaks()
     rows, classes, kernels = [], [], []
     for width in (1024, 2048):
-        for label, cfg_dict in ((f"Zikevik-{width}", zikevik_config(width)), (f"Pikasun-{width}", pikasun_config(width))):
+        for label, cfg_dict in models_at(width):
             cfg = config_from_dict(cfg_dict)
-            with tempfile.TemporaryDirectory(prefix="bench_zikevik_") as d:
+            with tempfile.TemporaryDirectory(prefix="bench_beside_") as d:
                 z.write_random_model(cfg, 0, d)
                 eng = z.Engine(d, "bfloat16", max_num_seqs=64, max_batched_tokens=2048 + 64, max_model_len=CONTEXT,
                                max_tokens=64 * CONTEXT, page_size=args.page_size)
@@ -844,7 +846,7 @@ def run_zikevik(args):
                 print(json.dumps(classes[-1]), flush=True)
                 del eng
                 torch.cuda.empty_cache()
-        kernels += zikevik_kernel_rooflines(width, hbm_peak, flops_peak)
+        kernels += kernel_rooflines(width, hbm_peak, flops_peak)
     for r in kernels:
         print(json.dumps(r), flush=True)
     print(f"\npeaks ({peak_src}): {hbm_peak:.0f} GB/s copy bandwidth, {flops_peak:.0f} TFLOP/s bf16 product (burst)\n")
@@ -853,12 +855,19 @@ def run_zikevik(args):
     for r in rows:
         print(f"| {r['model']} | {r['point']} | {r['ms']} | {r['tokens_per_s']} | {r.get('e2e_tokens_per_s', '')} | "
               f"{r.get('frac_of_copy_peak', '')} | {r.get('launches_per_step', '')} |")
-    print("\n| kernel | point | width | us | GFLOP | TFLOP/s | of the tensor peak | MB | GB/s | of the copy peak |")
-    print("|---|---|---|---|---|---|---|---|---|---|")
+    print("\n| kernel | point | width | us | GFLOP | TFLOP/s | of the tensor peak | MB | GB/s | of the copy peak | times the roofline |")
+    print("|---|---|---|---|---|---|---|---|---|---|---|")
     for r in kernels:
         print(f"| {r['kernel']} | {r['point']} | {r['width']} | {r['us']} | {r['GFLOP']} | {r['TFLOP_per_s']} | {r['of_tensor_peak']} | "
-              f"{r['MB']} | {r['GB_per_s']} | {r['of_copy_peak']} |")
+              f"{r['MB']} | {r['GB_per_s']} | {r['of_copy_peak']} | {r.get('distance', '')} |")
     return 0
+
+
+def run_zikevik(args):
+    """Prefill and decode throughput of the Zikevik design at two widths beside the Pikasun design (the closest one:
+    latent attention in front of gated feed-forwards) of the same width, layer count and vocabulary; the time of a prefill
+    and of a decode step by kernel class; and its kernels alone beside the like kernels.  JSON lines, then markdown."""
+    return run_beside(args, lambda w: ((f"Zikevik-{w}", zikevik_config(w)), (f"Pikasun-{w}", pikasun_config(w))), zikevik_kernel_rooflines)
 
 
 def lolivik_config(width, layers=16, vocab=65536):
@@ -995,61 +1004,155 @@ def run_lolivik(args):
     recurrent mixer and attention with a sink in front of dense feed-forwards and routed experts) of the same width, layer
     count and vocabulary; the time of a prefill and of a decode step by kernel class; and its kernels alone beside the like
     kernels.  JSON lines, then markdown."""
+    return run_beside(args, lambda w: ((f"Lolivik-{w}", lolivik_config(w)), (f"Zikevik-{w}", zikevik_config(w))), lolivik_kernel_rooflines)
+
+
+def sogenex_config(width, layers=16, vocab=65536):
+    """A Sogenex model of a real model's proportions: groups of four layers (three state-space mixers and windowed differential
+    attention, each in front of eight experts of which a token uses two, with a gated unit for every token; one of the
+    state-space mixers has no feed-forward).  The recurrence is twice the model's width in heads of 64 with 128 states; the
+    attention's two maps have size 64 over values of 128, four query heads a key/value head, a window of 1024."""
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 2 * width // 512, "conv": 4, "norm_groups": 2 * width // 512}
+    att = {"heads": width // 128, "kv_heads": width // 512, "dim": 64, "vdim": 128, "scale": 0.125, "mask": {"size": 1024}, "diff": 0.5}
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 2}, "router": {"experts": 8, "top": 2}, "shared": {"ff": 3 * width // 2}}
+    group = [("mamba2", ssm, moe), ("attention", att, moe), ("mamba2", ssm, None), ("mamba2", ssm, moe)]
+    return {"architecture": "Sogenex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0,
+            "layers": [{"type": t, "mixer": dict(m), "mlp": f and dict(f)} for t, m, f in (group[i % 4] for i in range(layers))]}
+
+
+def sogenex_kernel_rooflines(width, hbm_peak, flops_peak):
+    """Every kernel that the design adds, alone at the sizes of `sogenex_config(width)`, beside the like kernel of an existing
+    design: the state-space recurrence (with its convolution, gate and norm) beside the matrix memory with the same state
+    (Lolivik's); the two maps of windowed differential attention beside windowed grouped-query attention (LFM2's kernels, and
+    Lolivik's with kept first positions) with as many key and query values, and with heads of the size that the maps' values have; the experts without a gate and their
+    gated unit beside Lolivik's bounded experts and unit with as many parameters a token; the embedding with position vectors
+    beside the one without.  A portion of 2048 tokens and 64 single tokens over contexts of 2048, timed with CUDA events, the
+    L2 flushed before every call; `distance` is the time over the larger of the two roofline times."""
     import torch
-    import zig_ai_b200 as z
-    from zig_ai_b200.config import config_from_dict
-    hbm_peak, flops_peak, peak_src = peaks()
-    rows, classes, kernels = [], [], []
-    for width in (1024, 2048):
-        for label, cfg_dict in ((f"Lolivik-{width}", lolivik_config(width)), (f"Zikevik-{width}", zikevik_config(width))):
-            cfg = config_from_dict(cfg_dict)
-            with tempfile.TemporaryDirectory(prefix="bench_lolivik_") as d:
-                z.write_random_model(cfg, 0, d)
-                eng = z.Engine(d, "bfloat16", max_num_seqs=64, max_batched_tokens=2048 + 64, max_model_len=CONTEXT,
-                               max_tokens=64 * CONTEXT, page_size=args.page_size)
-                nums = engine_numbers(eng)
-                active = params_read(nums, 1)
-                prefill_ms = time_prefill(eng, reps=5)
-                T = PREFILL_TOKENS
-                rows.append({"model": label, "width": width, "matrix_params_M": round(nums["matrix_params"] / 1e6, 1),
-                             "active_params_M": round(active / 1e6, 1), "point": "prefill 2048", "ms": round(prefill_ms, 3),
-                             "tokens_per_s": round(T / prefill_ms * 1e3),
-                             "matrix_TFLOP_per_s": round(2 * T * active / prefill_ms / 1e9, 1)})
-                print(json.dumps(rows[-1]), flush=True)
-                for B in (1, 8, 64):
-                    dev_ms, e2e_ms, ctx_tokens, launches, _, _, _ = time_decode(eng, B, max(min(args.steps, 100), 20), args.warmup)
-                    read = params_read(nums, B)       # of the experts, a step reads those that its tokens chose
-                    step_bytes = 2 * read + ctx_tokens * nums["kv_bytes_per_token"] + 2 * B * nums["state_bytes"]
-                    rows.append({"model": label, "width": width, "point": f"decode batch {B}", "ms": round(dev_ms, 4),
-                                 "e2e_ms": round(e2e_ms, 4), "tokens_per_s": round(B / dev_ms * 1e3),
-                                 "e2e_tokens_per_s": round(B / e2e_ms * 1e3), "GB_a_step": round(step_bytes / 1e9, 3),
-                                 "frac_of_copy_peak": round(step_bytes / (dev_ms * 1e-3) / 1e9 / hbm_peak, 3),
-                                 "launches_per_step": round(launches)})
-                    print(json.dumps(rows[-1]), flush=True)
-                g = random.Random(5)
-                V = eng.config.vocab_size
-                eng.flush()
-                pre = kernel_classes(eng, [("kc", [g.randrange(V) for _ in range(T)], [T - 1])])
-                dec = kernel_classes(eng, [(f"kc{i}", [g.randrange(V)], [0]) for i in range(64)])
-                classes.append({"model": label, "prefill_2048_ms_by_class": pre, "decode_64_first_token_ms_by_class": dec})
-                print(json.dumps(classes[-1]), flush=True)
-                del eng
-                torch.cuda.empty_cache()
-        kernels += lolivik_kernel_rooflines(width, hbm_peak, flops_peak)
-    for r in kernels:
-        print(json.dumps(r), flush=True)
-    print(f"\npeaks ({peak_src}): {hbm_peak:.0f} GB/s copy bandwidth, {flops_peak:.0f} TFLOP/s bf16 product (burst)\n")
-    print("| model | point | ms a step (device) | tokens/s (device) | tokens/s (end to end) | of the copy peak | launches a step |")
-    print("|---|---|---|---|---|---|---|")
-    for r in rows:
-        print(f"| {r['model']} | {r['point']} | {r['ms']} | {r['tokens_per_s']} | {r.get('e2e_tokens_per_s', '')} | "
-              f"{r.get('frac_of_copy_peak', '')} | {r.get('launches_per_step', '')} |")
-    print("\n| kernel | point | width | us | GFLOP | TFLOP/s | of the tensor peak | MB | GB/s | of the copy peak |")
-    print("|---|---|---|---|---|---|---|---|---|---|")
-    for r in kernels:
-        print(f"| {r['kernel']} | {r['point']} | {r['width']} | {r['us']} | {r['GFLOP']} | {r['TFLOP_per_s']} | {r['of_tensor_peak']} | "
-              f"{r['MB']} | {r['GB_per_s']} | {r['of_copy_peak']} |")
-    return 0
+    from zig_ai_b200.cache.manager import CacheView
+    from zig_ai_b200.engine.batch import pack_step
+    from zig_ai_b200.kernels import ops
+    ops.require(torch.bfloat16, ("attention", "attention_mma", "attention_tma", "attention_tc", "attention_difference", "mamba2", "mlstm",
+                                 "causal_conv", "moe", "gemm_tc"))
+    dev, dt = torch.device("cuda"), torch.bfloat16
+    ps, D, V = 64, 64, 128
+    Ha, Ga = width // 128, width // 512
+    Hm, Gm, Ns, Vm = 2 * width // 64, 2 * width // 512, 128, 64
+    E, top, F = 8, 2, 3 * width // 2
+    g = torch.Generator().manual_seed(1)
+    rnd = lambda *shape, s=1.0: (torch.randn(*shape, generator=g) * s).to(dt).to(dev)
+    rows = []
+
+    def step_of(ctx, q_lens):
+        spans, tables, at = [], [], 1
+        width_pages = max(-(-(c + n) // ps) for c, n in zip(ctx, q_lens))
+        for s_, (c, n) in enumerate(zip(ctx, q_lens)):
+            need = -(-(c + n) // ps)
+            tables.append(list(range(at, at + need)) + [0] * (width_pages - need))
+            at += need
+            spans.append((s_, c, [0] * n, [], s_ + 1))
+        return pack_step(ops, dt, dev, spans, {0: tables}), at
+
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=10):
+        for _ in range(3):
+            fn()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        total = 0.0
+        for _ in range(reps):
+            flush.zero_()                                    # larger than L2: the timed call starts cold
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            total += a.elapsed_time(b)
+        return total / reps
+
+    for point, ctx, q_lens in (("2048-token portion", [0], [2048]), ("64 single tokens, context 2048", [2047] * 64, [1] * 64)):
+        step, n_pages = step_of(ctx, q_lens)
+        N, B = sum(q_lens), len(q_lens)
+        # the recurrences, from the projections' rows to the output projection's input
+        I, ch = Hm * Vm, Hm * Vm + 2 * Gm * Ns
+        y = rnd(N, I + ch + Hm)
+        vec = lambda n, v=0.0: torch.full((n,), v, device=dev)
+        taps, state, hist = torch.randn(ch, 4, generator=g).to(dev), torch.zeros(B + 1, Hm, Ns, Vm, device=dev), torch.zeros(B + 1, 3, ch, device=dev)
+        by = N * (2 * I + ch + Hm) * 2 + B * (Hm * Ns * Vm + 3 * ch) * 8
+        rows.append(("state-space recurrence: convolution, state, gate, norm", point, timed(lambda: ops.mamba2(
+            y, (0, I, I + ch), taps, vec(ch), vec(Hm), vec(Hm), vec(Hm, 1.0), vec(I, 1.0), 1e-6, Gm, state, hist, step, Hm, Gm, Ns, Vm)),
+            4.0 * N * Hm * Ns * Vm, by))
+        at, cols = [], 0
+        for n in (Hm * Ns, Hm * Ns, I, I, Hm, Hm):
+            at.append(cols)
+            cols += -(-n // 8) * 8
+        ym, mstate = rnd(N, cols), torch.zeros(B + 1, Hm, Ns + 1, Vm + 1, device=dev)
+        rows.append(("matrix memory with log gates, the same state (Lolivik's)", point, timed(lambda: ops.mlstm(
+            ym, at, vec(Hm), vec(Hm), 15.0, vec(I, 1.0), 1e-6, mstate, step, Hm, Ns, Vm)), 4.0 * N * Hm * Ns * Vm,
+            N * (cols + I) * 2 + B * Hm * Ns * Vm * 8))
+        del ym
+        # attention: (query, key) pairs seen; two maps of D over values of V
+        pairs = sum(sum(min(c + i + 1, 1024) for i in range(n)) for c, n in zip(ctx, q_lens))
+        cached = sum(min(c + n, 1023 + n) for c, n in zip(ctx, q_lens))
+        view = CacheView(0, rnd(n_pages, 2, Ga, ps, V, s=0.5), step.block_tables[0], ps)
+        qkv = rnd(N, (2 * Ha + 2 * Ga) * V)
+        maps = qkv[:, :2 * Ha * V].reshape(N, Ha, 2, 2, D)
+        maps[:, :, 0, 1] = 0
+        maps[:, :, 1, 0] = 0
+
+        def plain(view, qkv, H, G, Dh):
+            if N == B:
+                return lambda: ops.decode_attention_fused(qkv, None, None, 0.0, 0, 1.0, step, view, H, G, Dh, 0.125, 1024)
+            q = qkv[:, :H * Dh].contiguous()
+            return lambda: ops.paged_attention(q, step, view, H, G, Dh, 0.125, 1024)
+        two = plain(view, qkv, 2 * Ha, Ga, V)
+        fl, by = 2.0 * pairs * 2 * Ha * (D + V), cached * Ga * 2 * V * 2 + N * Ha * (2 * D + V) * 2
+        rows.append(("differential attention: two maps, their difference normed", point,
+                     timed(lambda: ops.attention_difference(two(), Ha, V, V, 0.5, 0.5, 1e-6)), fl, by))
+        rows.append(("windowed attention, heads of 128 (LFM2's kernels)", point, timed(two), 2.0 * pairs * 2 * Ha * 2 * V,
+                     cached * Ga * 2 * V * 2 + N * Ha * 4 * V * 2))
+        view64 = CacheView(0, rnd(n_pages, 2, 2 * Ga, ps, D, s=0.5), step.block_tables[0], ps)
+        qkv64 = rnd(N, (2 * Ha + 4 * Ga) * D)
+        rows.append(("windowed attention, heads of 64 (LFM2's kernels)", point, timed(plain(view64, qkv64, 2 * Ha, 2 * Ga, D)),
+                     2.0 * pairs * 2 * Ha * 2 * D, cached * 2 * Ga * 2 * D * 2 + N * Ha * 4 * D * 2))
+        q64 = qkv64[:, :2 * Ha * D].contiguous()
+        rows.append(("windowed attention, first positions kept, heads of 64 (Lolivik's)", point, timed(lambda: ops.paged_attention(
+            q64, step, view64, 2 * Ha, 2 * Ga, D, 0.125, 1024, keep_first=4)), 2.0 * pairs * 2 * Ha * 2 * D,
+            cached * 2 * Ga * 2 * D * 2 + N * Ha * 4 * D * 2))
+        # the feed-forwards: a token's two experts and its unit
+        x = rnd(N, width)
+        w_router, r_bias = (torch.randn(E + 1, width, generator=g) * 0.05).to(dev), vec(E)
+        w_up, w_dn = rnd(E, F, width, s=0.02), rnd(E, width, F, s=0.02)
+        s_up, s_dn = rnd(F, width, s=0.02), rnd(width, F, s=0.02)
+        used = min(E, N * top)
+        fl, by = 2.0 * N * (top + 1) * 2 * width * F, (used + 1) * 2 * width * F * 2 + N * width * 4
+        unit = lambda: ops.linear(ops.linear_activation(x, s_up, "relu2"), s_dn)
+        rows.append((f"experts without a gate ({top} of {E}) and the gated unit", point, timed(lambda: ops.routed_experts(
+            x, w_router, w_up, w_dn, top, False, "output", score="chosen", act="relu2", router_bias=r_bias, unit=unit(), unit_gated=True)), fl, by))
+        F2 = width
+        l_gu, l_dn = rnd(E, 2 * F2, width, s=0.02), rnd(E, width, F2, s=0.02)
+        u_gu, u_dn = rnd(2 * F2, width, s=0.02), rnd(width, F2, s=0.02)
+        w8 = w_router[:E].contiguous()
+        bounded = lambda: ops.weighted_sum(
+            ops.routed_experts(x, w8, l_gu, l_dn, top, True, "output", score="softmax", act="clamped", limit=7.0, alpha=1.702),
+            ops.linear(ops.linear_clamped_glu(x, u_gu, F2, 7.0, 1.702), u_dn), 1.0, 1.0)
+        rows.append((f"bounded experts ({top} of {E}) and their unit (Lolivik's)", point, timed(bounded), fl, by))
+        rows.append(("the unit alone: relu squared", point, timed(unit), 2.0 * N * 2 * width * F, 2 * width * F * 2 + N * width * 4))
+        rows.append(("a bounded gated unit alone (Lolivik's)", point, timed(lambda: ops.linear(ops.linear_clamped_glu(x, u_gu, F2, 7.0, 1.702), u_dn)),
+                     2.0 * N * 2 * width * F, 2 * width * F * 2 + N * width * 4))
+        ids, table = torch.randint(0, 65536, (N,), generator=g).to(torch.int32).to(dev), rnd(65536, width)
+        rows.append(("embedding with position vectors", point, timed(lambda: ops.embed(ids, table, 1.0, step.positions)), 0.0, N * width * 6))
+        rows.append(("embedding (shared with LFM2)", point, timed(lambda: ops.embed(ids, table)), 0.0, N * width * 6))
+    return [{"kernel": k, "point": p, "width": width, "us": round(ms * 1e3, 2), "GFLOP": round(fl / 1e9, 2), "MB": round(by / 1e6, 2),
+             "TFLOP_per_s": round(fl / ms / 1e9, 1), "of_tensor_peak": round(fl / ms / 1e9 / flops_peak, 4),
+             "GB_per_s": round(by / ms / 1e6, 1), "of_copy_peak": round(by / ms / 1e6 / hbm_peak, 4),
+             "distance": round(ms / max(fl / 1e9 / flops_peak, by / 1e6 / hbm_peak), 2)} for k, p, ms, fl, by in rows]
+
+
+def run_sogenex(args):
+    """Prefill and decode throughput of the Sogenex design at two widths beside the Lolivik design (the closest one: a recurrence
+    over a matrix state and windowed attention in front of routed experts with a shared unit) of the same width, layer count and
+    vocabulary; the time of a prefill and of a decode step by kernel class; and its kernels alone beside the like kernels."""
+    return run_beside(args, lambda w: ((f"Sogenex-{w}", sogenex_config(w)), (f"Lolivik-{w}", lolivik_config(w))), sogenex_kernel_rooflines)
 
 
 def run_table(args):
@@ -1405,9 +1508,9 @@ def main():
     ap.add_argument("--steps", type=int, default=200)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "gemm", "timeline", "table", "stream", "long", "sample", "vunolorn", "pikasun", "zikevik", "lolivik"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "gemm", "timeline", "table", "stream", "long", "sample", "vunolorn", "pikasun", "zikevik", "lolivik", "sogenex"],
                     help="profiling aid: run only the batch-8 decode steps or only the prefill (prints a short line); "
-                         "table: every figure of the 350M, 700M and 1.2B shapes (profiles/measurements.md); pikasun: the Pikasun design beside LFM2 at equal width; zikevik: the Zikevik design beside Pikasun at equal width, and its kernels beside the like ones; lolivik: the Lolivik design beside Zikevik at equal width, and its kernels beside the like ones; vunolorn: the "
+                         "table: every figure of the 350M, 700M and 1.2B shapes (profiles/measurements.md); pikasun: the Pikasun design beside LFM2 at equal width; zikevik: the Zikevik design beside Pikasun at equal width, and its kernels beside the like ones; lolivik: the Lolivik design beside Zikevik at equal width, and its kernels beside the like ones; sogenex: the Sogenex design beside Lolivik, likewise; vunolorn: the "
                          "Vunolorn hybrid at two widths beside LFM2 at equal width, and its recurrent kernels alone")
     ap.add_argument("--batch", type=int, default=8, help="with --only decode: the batch size; with --only stream: 24, 64 or "
                                                          "128 runs that row count only")

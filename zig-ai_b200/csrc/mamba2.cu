@@ -143,27 +143,33 @@ __device__ __forceinline__ bool m2_find_chunk(const Mamba2Args& a, int b, int& s
     return false;
 }
 
-// The chunk's step sizes d_j and the running sums L_j of a d (both 64 values; rows beyond the chunk have d = 0), by the first
-// 64 threads of the block; everyone calls it.
-__device__ __forceinline__ void m2_decays(const Mamba2Args& a, int h, int t0, int t1, float* s_d, float* s_l) {
+// The chunk's step sizes d_j and the running sums L_j of a d, in units of ln 2 (both 64 values; rows beyond the chunk have
+// d = 0), by the first 64 threads of the block; everyone calls it.  The sums are made in 64-bit and kept as two 32-bit numbers
+// each, so that a difference of two of them is good to the last bits whatever the chunk's rows before it have summed up to.
+__device__ __forceinline__ void m2_decays(const Mamba2Args& a, int h, int t0, int t1, float* s_d, float2* s_l, double* s_carry) {
     const int j = threadIdx.x, lane = threadIdx.x & 31;
-    float l = 0.f;
+    double l = 0.0;
     if (j < M2_Q) {
         float d = 0.f;
         if (t0 + j < t1) d = m2_softplus(to_float(((const bf16*)a.dt)[(size_t)(t0 + j) * a.dt_stride + h]) + a.dt_bias[h]);
         s_d[j] = d;
-        l = -expf(a.a_log[h]) * d;
+        l = -1.4426950408889634 * (double)(expf(a.a_log[h]) * d);
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
-            const float up = __shfl_up_sync(0xffffffffu, l, o);
+            const double up = __shfl_up_sync(0xffffffffu, l, o);
             if (lane >= o) l += up;
         }
-        s_l[j] = l;
+        if (j == 31) *s_carry = l;
     }
     __syncthreads();
-    if (j >= 32 && j < M2_Q) s_l[j] = l + s_l[31];
+    if (j < M2_Q) {
+        if (j >= 32) l += *s_carry;
+        const float hi = (float)l;
+        s_l[j] = make_float2(hi, (float)(l - (double)hi));
+    }
     __syncthreads();
 }
+__device__ __forceinline__ float m2_between(float2 later, float2 earlier) { return (later.x - earlier.x) + (later.y - earlier.y); }
 
 // rows t0.. of a column slice of u into shared memory [M2_Q][ld] (zeros beyond the chunk and beyond `cols` up to `cols_p`)
 __device__ __forceinline__ void m2_load_rows(bf16* dst, int ld, const Mamba2Args& a, int at, int cols, int cols_p, int t0, int t1) {
@@ -191,13 +197,25 @@ __device__ __forceinline__ void m2_split(float v, float& hi, float& mid, float& 
     mid = __bfloat162float(__float2bfloat16_rn(r));
     lo = r - mid;
 }
+// two neighbouring values, each split: p[k] holds the k-th parts
+__device__ __forceinline__ void m2_split2(float v0, float v1, uint32_t (&p)[3]) {
+    float a0, a1, a2, b0, b1, b2;
+    m2_split(v0, a0, a1, a2);
+    m2_split(v1, b0, b1, b2);
+    p[0] = pack_bf16(a0, b0);
+    p[1] = pack_bf16(a1, b1);
+    p[2] = pack_bf16(a2, b2);
+}
 
-// pass 1: ends [chunk, H, N, V] and last [chunk, H] (the chunk's L_last).  VT columns of V a block.
+// pass 1: ends [chunk, H, N, V] and last [chunk, H] (the chunk's L_last).  VT columns of V a block; eight warps, each in turn
+// 16 states x 32 columns.
 template <int VT>
-__global__ void __launch_bounds__(128) mamba2_chunk_state_kernel(const Mamba2Args a, float* __restrict__ ends, float* __restrict__ last) {
+__global__ void __launch_bounds__(256) mamba2_chunk_state_kernel(const Mamba2Args a, float* __restrict__ ends, float* __restrict__ last) {
     extern __shared__ __align__(16) unsigned char m2_raw[];
-    __shared__ float s_d[M2_Q], s_l[M2_Q];
-    constexpr int LDX = VT + M2_PAD;
+    __shared__ float s_d[M2_Q], s_w[M2_Q];
+    __shared__ float2 s_l[M2_Q];
+    __shared__ double s_carry;
+    constexpr int LDX = VT + M2_PAD, VW = 32, VG = VT / VW;
     const int np = (a.N + 15) & ~15, ldb = np + M2_PAD;
     bf16* sb = reinterpret_cast<bf16*>(m2_raw);              // [Q][ldb]
     bf16* sx = sb + M2_Q * ldb;                              // [3][Q][LDX]
@@ -206,29 +224,36 @@ __global__ void __launch_bounds__(128) mamba2_chunk_state_kernel(const Mamba2Arg
     int seq, t0, t1;
     if (!m2_find_chunk(a, blockIdx.x, seq, t0, t1)) return;
     const int h = blockIdx.y, g = h / (a.H / a.G), v0 = blockIdx.z * VT, nv = min(VT, a.V - v0);
-    m2_load_rows(sb, ldb, a, a.H * a.V + g * a.N, a.N, np, t0, t1);
     m2_load_rows(sx, LDX, a, h * a.V + v0, nv, VT, t0, t1);
     cp_async_commit();
-    m2_decays(a, h, t0, t1, s_d, s_l);
-    cp_async_wait<0>();
+    m2_load_rows(sb, ldb, a, a.H * a.V + g * a.N, a.N, np, t0, t1);
+    cp_async_commit();
+    m2_decays(a, h, t0, t1, s_d, s_l, &s_carry);
+    if (threadIdx.x < M2_Q) s_w[threadIdx.x] = exp2f(m2_between(s_l[M2_Q - 1], s_l[threadIdx.x])) * s_d[threadIdx.x];
+    if (threadIdx.x == 0 && v0 == 0) last[(size_t)blockIdx.x * a.H + h] = s_l[M2_Q - 1].x;
+    cp_async_wait<1>();
     __syncthreads();
-    const float l_last = s_l[M2_Q - 1];
-    if (threadIdx.x == 0 && v0 == 0) last[(size_t)blockIdx.x * a.H + h] = l_last;
-    for (int i = threadIdx.x; i < M2_Q * VT; i += blockDim.x) {
-        const int j = i / VT, c = i % VT;
-        float hi, mid, lo;
-        m2_split(__bfloat162float(sx[j * LDX + c]) * (expf(l_last - s_l[j]) * s_d[j]), hi, mid, lo);
-        sx[j * LDX + c] = __float2bfloat16_rn(hi);
-        sx[(M2_Q + j) * LDX + c] = __float2bfloat16_rn(mid);
-        sx[(2 * M2_Q + j) * LDX + c] = __float2bfloat16_rn(lo);
+#pragma unroll
+    for (int i = threadIdx.x; i < M2_Q * VT / 2; i += 256) {
+        const int j = i / (VT / 2), c = (i % (VT / 2)) * 2;
+        uint32_t* p = reinterpret_cast<uint32_t*>(sx + j * LDX + c);
+        const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        const float w = s_w[j];
+        uint32_t q[3];
+        m2_split2(x.x * w, x.y * w, q);
+        p[0] = q[0];
+        p[M2_Q * LDX / 2] = q[1];
+        p[M2_Q * LDX] = q[2];
     }
+    cp_async_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, r8 = lane & 7;
     float* e = ends + ((size_t)blockIdx.x * a.H + h) * a.N * a.V;
-    for (int mt = warp; mt < np / 16; mt += 4) {             // 16 states a time
-        float acc[VT / 8][4];
+    for (int item = warp; item < np / 16 * VG; item += 8) {
+        const int mt = item / VG, vb = (item % VG) * VW;
+        float acc[VW / 8][4];
 #pragma unroll
-        for (int i = 0; i < VT / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+        for (int i = 0; i < VW / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
         for (int ks = 0; ks < M2_Q / 16; ++ks) {
             uint32_t fa[4];
@@ -236,9 +261,9 @@ __global__ void __launch_bounds__(128) mamba2_chunk_state_kernel(const Mamba2Arg
 #pragma unroll
             for (int p = 2; p >= 0; --p) {                   // the small parts first
 #pragma unroll
-                for (int vp = 0; vp < VT / 16; ++vp) {
+                for (int vp = 0; vp < VW / 16; ++vp) {
                     uint32_t fb[4];
-                    ldmatrix_x4_trans(fb, sx + (p * M2_Q + ks * 16 + (mi & 1) * 8 + r8) * LDX + vp * 16 + (mi >> 1) * 8);
+                    ldmatrix_x4_trans(fb, sx + (p * M2_Q + ks * 16 + (mi & 1) * 8 + r8) * LDX + vb + vp * 16 + (mi >> 1) * 8);
                     mma_bf16(acc[2 * vp], fa, fb[0], fb[1]);
                     mma_bf16(acc[2 * vp + 1], fa, fb[2], fb[3]);
                 }
@@ -247,8 +272,8 @@ __global__ void __launch_bounds__(128) mamba2_chunk_state_kernel(const Mamba2Arg
         const int n = mt * 16 + (lane >> 2), tq = lane & 3;
         const bool even = ((a.V | v0) & 1) == 0;
 #pragma unroll
-        for (int i = 0; i < VT / 8; ++i) {
-            const int c = i * 8 + 2 * tq;
+        for (int i = 0; i < VW / 8; ++i) {
+            const int c = vb + i * 8 + 2 * tq;
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
                 const int nn = n + 8 * half;
@@ -303,7 +328,7 @@ __global__ void __launch_bounds__(128) mamba2_state_pass_kernel(const Mamba2Args
             float* p = ends + (size_t)(c0 + c + i) * HNV + idx;
             if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(S[0], S[1], S[2], S[3]);
             else *p = S[0];
-            const float keep = expf(l[i]);
+            const float keep = exp2f(l[i]);
 #pragma unroll
             for (int k = 0; k < VEC; ++k) S[k] = fmaf(keep, S[k], e[i][k]);
         }
@@ -314,12 +339,14 @@ __global__ void __launch_bounds__(128) mamba2_state_pass_kernel(const Mamba2Args
     }
 }
 
-// pass 3: starts [chunk, H, N, V] is the state before every chunk.  Four warps, 16 rows each.
+// pass 3: starts [chunk, H, N, V] is the state before every chunk.  Eight warps: 16 rows x half of the columns each.
 template <int VT>
-__global__ void __launch_bounds__(128) mamba2_chunk_out_kernel(const Mamba2Args a, const float* __restrict__ starts) {
+__global__ void __launch_bounds__(256) mamba2_chunk_out_kernel(const Mamba2Args a, const float* __restrict__ starts) {
     extern __shared__ __align__(16) unsigned char m2_raw[];
-    __shared__ float s_d[M2_Q], s_l[M2_Q];
-    constexpr int LDX = VT + M2_PAD;
+    __shared__ float s_d[M2_Q];
+    __shared__ float2 s_l[M2_Q];
+    __shared__ double s_carry;
+    constexpr int LDX = VT + M2_PAD, VW = VT / 2;
     const int np = (a.N + 15) & ~15, ldb = np + M2_PAD;
     bf16* sc = reinterpret_cast<bf16*>(m2_raw);              // [Q][ldb]
     bf16* sb = sc + M2_Q * ldb;                              // [Q][ldb]
@@ -336,21 +363,27 @@ __global__ void __launch_bounds__(128) mamba2_chunk_out_kernel(const Mamba2Args 
     cp_async_commit();
     const float* S = starts + ((size_t)blockIdx.x * a.H + h) * a.N * a.V + v0;
     if ((a.V & 3) == 0 && (nv & 3) == 0) {
-        for (int i = threadIdx.x; i < np * (VT / 4); i += blockDim.x) {
-            const int n = i / (VT / 4), c = (i % (VT / 4)) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (n < a.N && c < nv) v = *reinterpret_cast<const float4*>(S + (size_t)n * a.V + c);
-            float p[3][4];
-            m2_split(v.x, p[0][0], p[1][0], p[2][0]);
-            m2_split(v.y, p[0][1], p[1][1], p[2][1]);
-            m2_split(v.z, p[0][2], p[1][2], p[2][2]);
-            m2_split(v.w, p[0][3], p[1][3], p[2][3]);
+        constexpr int PER = VT / 4, U = 4;                   // four loads in flight a thread
+        for (int i0 = threadIdx.x; i0 < np * PER; i0 += 256 * U) {
+            float4 v[U];
 #pragma unroll
-            for (int k = 0; k < 3; ++k)
-                *reinterpret_cast<uint2*>(ss + (k * np + n) * LDX + c) = make_uint2(pack_bf16(p[k][0], p[k][1]), pack_bf16(p[k][2], p[k][3]));
+            for (int k = 0; k < U; ++k) {
+                const int i = i0 + 256 * k, n = i / PER, c = (i % PER) * 4;
+                v[k] = (n < a.N && c < nv) ? *reinterpret_cast<const float4*>(S + (size_t)n * a.V + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int k = 0; k < U; ++k) {
+                const int i = i0 + 256 * k, n = i / PER, c = (i % PER) * 4;
+                if (n >= np) continue;
+                uint32_t p[3], q[3];
+                m2_split2(v[k].x, v[k].y, p);
+                m2_split2(v[k].z, v[k].w, q);
+#pragma unroll
+                for (int m = 0; m < 3; ++m) *reinterpret_cast<uint2*>(ss + (m * np + n) * LDX + c) = make_uint2(p[m], q[m]);
+            }
         }
     } else {
-        for (int i = threadIdx.x; i < np * VT; i += blockDim.x) {
+        for (int i = threadIdx.x; i < np * VT; i += 256) {
             const int n = i / VT, c = i % VT;
             float hi, mid, lo;
             m2_split((n < a.N && c < nv) ? S[(size_t)n * a.V + c] : 0.f, hi, mid, lo);
@@ -359,25 +392,27 @@ __global__ void __launch_bounds__(128) mamba2_chunk_out_kernel(const Mamba2Args 
             ss[(2 * np + n) * LDX + c] = __float2bfloat16_rn(lo);
         }
     }
-    m2_decays(a, h, t0, t1, s_d, s_l);
+    m2_decays(a, h, t0, t1, s_d, s_l, &s_carry);
     cp_async_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mi = lane >> 3, r8 = lane & 7;
-    const int i0 = warp * 16, ra = i0 + (lane >> 2), rb = ra + 8, tq = lane & 3;
-    const float la = s_l[ra], lb = s_l[rb];
+    const int wr = warp & 3, vb = (warp >> 2) * VW;
+    const int i0 = wr * 16, ra = i0 + (lane >> 2), rb = ra + 8, tq = lane & 3;
+    const float2 la = s_l[ra], lb = s_l[rb];
 
     // scores C . B of this warp's rows with the rows up to its own last one, and the read-out of the state before the chunk
-    float sco[M2_Q / 8][4], acc[VT / 8][4];
+    float sco[M2_Q / 8][4], acc[VW / 8][4];
 #pragma unroll
     for (int i = 0; i < M2_Q / 8; ++i) sco[i][0] = sco[i][1] = sco[i][2] = sco[i][3] = 0.f;
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int i = 0; i < VW / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll 2
     for (int ks = 0; ks < np / 16; ++ks) {
         uint32_t fa[4];
         ldmatrix_x4(fa, sc + (i0 + (mi & 1) * 8 + r8) * ldb + ks * 16 + (mi >> 1) * 8);
 #pragma unroll
         for (int jp = 0; jp < M2_Q / 16; ++jp) {
-            if (jp > warp) continue;
+            if (jp > wr) continue;
             uint32_t fb[4];
             ldmatrix_x4(fb, sb + (jp * 16 + (mi >> 1) * 8 + r8) * ldb + ks * 16 + (mi & 1) * 8);
             mma_bf16(sco[2 * jp], fa, fb[0], fb[1]);
@@ -386,44 +421,43 @@ __global__ void __launch_bounds__(128) mamba2_chunk_out_kernel(const Mamba2Args 
 #pragma unroll
         for (int p = 2; p >= 0; --p) {
 #pragma unroll
-            for (int vp = 0; vp < VT / 16; ++vp) {
+            for (int vp = 0; vp < VW / 16; ++vp) {
                 uint32_t fb[4];
-                ldmatrix_x4_trans(fb, ss + (p * np + ks * 16 + (mi & 1) * 8 + r8) * LDX + vp * 16 + (mi >> 1) * 8);
+                ldmatrix_x4_trans(fb, ss + (p * np + ks * 16 + (mi & 1) * 8 + r8) * LDX + vb + vp * 16 + (mi >> 1) * 8);
                 mma_bf16(acc[2 * vp], fa, fb[0], fb[1]);
                 mma_bf16(acc[2 * vp + 1], fa, fb[2], fb[3]);
             }
         }
     }
-    const float ea = expf(la), eb = expf(lb);
+    const float ea = exp2f(la.x), eb = exp2f(lb.x);
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i) {
+    for (int i = 0; i < VW / 8; ++i) {
         acc[i][0] *= ea; acc[i][1] *= ea; acc[i][2] *= eb; acc[i][3] *= eb;
     }
     // the chunk's own rows
 #pragma unroll
     for (int ks = 0; ks < M2_Q / 16; ++ks) {
-        if (ks > warp) continue;
+        if (ks > wr) continue;
         uint32_t f[3][4];
 #pragma unroll
         for (int half = 0; half < 2; ++half) {               // columns ks * 16 + 8 half + 2 tq, + 1
             const int j = ks * 16 + 8 * half + 2 * tq;
-            const float d0 = s_d[j], d1 = s_d[j + 1], l0 = s_l[j], l1 = s_l[j + 1];
+            const float d0 = s_d[j], d1 = s_d[j + 1];
+            const float2 l0 = s_l[j], l1 = s_l[j + 1];
             const float* g4 = sco[2 * ks + half];
-            const float m[4] = {j <= ra ? g4[0] * (expf(la - l0) * d0) : 0.f, j + 1 <= ra ? g4[1] * (expf(la - l1) * d1) : 0.f,
-                                j <= rb ? g4[2] * (expf(lb - l0) * d0) : 0.f, j + 1 <= rb ? g4[3] * (expf(lb - l1) * d1) : 0.f};
-            float p[3][4];
-#pragma unroll
-            for (int k = 0; k < 4; ++k) m2_split(m[k], p[0][k], p[1][k], p[2][k]);
+            uint32_t p[3], q[3];
+            m2_split2(j <= ra ? g4[0] * (fast_exp2(m2_between(la, l0)) * d0) : 0.f, j + 1 <= ra ? g4[1] * (fast_exp2(m2_between(la, l1)) * d1) : 0.f, p);
+            m2_split2(j <= rb ? g4[2] * (fast_exp2(m2_between(lb, l0)) * d0) : 0.f, j + 1 <= rb ? g4[3] * (fast_exp2(m2_between(lb, l1)) * d1) : 0.f, q);
 #pragma unroll
             for (int k = 0; k < 3; ++k) {
-                f[k][2 * half] = pack_bf16(p[k][0], p[k][1]);
-                f[k][2 * half + 1] = pack_bf16(p[k][2], p[k][3]);
+                f[k][2 * half] = p[k];
+                f[k][2 * half + 1] = q[k];
             }
         }
 #pragma unroll
-        for (int vp = 0; vp < VT / 16; ++vp) {
+        for (int vp = 0; vp < VW / 16; ++vp) {
             uint32_t fb[4];
-            ldmatrix_x4_trans(fb, sx + (ks * 16 + (mi & 1) * 8 + r8) * LDX + vp * 16 + (mi >> 1) * 8);
+            ldmatrix_x4_trans(fb, sx + (ks * 16 + (mi & 1) * 8 + r8) * LDX + vb + vp * 16 + (mi >> 1) * 8);
 #pragma unroll
             for (int p = 2; p >= 0; --p) {
                 mma_bf16(acc[2 * vp], f[p], fb[0], fb[1]);
@@ -434,8 +468,8 @@ __global__ void __launch_bounds__(128) mamba2_chunk_out_kernel(const Mamba2Args 
     const float skip = a.skip[h];
     const bool even = ((a.V | v0) & 1) == 0;
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i) {
-        const int c = i * 8 + 2 * tq;
+    for (int i = 0; i < VW / 8; ++i) {
+        const int c = vb + i * 8 + 2 * tq;
         if (c >= nv) continue;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
@@ -470,8 +504,22 @@ __global__ void __launch_bounds__(256) mamba2_single_kernel(const Mamba2Args a, 
     const T* row = y_in + (size_t)s * stride;
     const float* hist = history + (size_t)slot * max(L - 1, 1) * ch;
     float* st = a.state + ((size_t)slot * a.H + h) * a.N * a.V;
-    // the first of this thread's state elements are asked for before the convolution
     const int lv = min((a.V + VEC - 1) / VEC, (int)blockDim.x), rg_n = blockDim.x / lv, vi = threadIdx.x % lv, rg = threadIdx.x / lv;
+    constexpr int U = 8;                         // rows of the state a thread has in flight
+    float S[U][VEC];
+    auto load = [&](int v, int n0) {
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int n = n0 + i * rg_n;
+            if (n >= a.N) continue;
+            const float* p = st + (size_t)n * a.V + v;
+            if constexpr (VEC == 4) {
+                const float4 q = *reinterpret_cast<const float4*>(p);
+                S[i][0] = q.x; S[i][1] = q.y; S[i][2] = q.z; S[i][3] = q.w;
+            } else S[i][0] = *p;
+        }
+    };
+    if (vi * VEC < a.V && rg < rg_n) load(vi * VEC, rg);      // (the first rows are on their way while the convolution runs)
     for (int i = threadIdx.x; i < a.V + 2 * a.N; i += blockDim.x) {
         const int c = i < a.V ? h * a.V + i : i < a.V + a.N ? inner + g * a.N + (i - a.V) : inner + (a.G + g) * a.N + (i - a.V - a.N);
         float acc = (conv_bias ? conv_bias[c] : 0.f) + taps[(size_t)c * L + (L - 1)] * to_float(row[xbc_at + c]);
@@ -492,19 +540,8 @@ __global__ void __launch_bounds__(256) mamba2_single_kernel(const Mamba2Args a, 
             x[k] = live ? d * sx[v + k] : 0.f;
             y[k] = 0.f;
         }
-        constexpr int U = 8;
         for (int n0 = rg; n0 < a.N && live; n0 += rg_n * U) {
-            float S[U][VEC];
-#pragma unroll
-            for (int i = 0; i < U; ++i) {
-                const int n = n0 + i * rg_n;
-                if (n >= a.N) continue;
-                const float* p = st + (size_t)n * a.V + v;
-                if constexpr (VEC == 4) {
-                    const float4 q = *reinterpret_cast<const float4*>(p);
-                    S[i][0] = q.x; S[i][1] = q.y; S[i][2] = q.z; S[i][3] = q.w;
-                } else S[i][0] = *p;
-            }
+            if (v0 > 0 || n0 > rg) load(v, n0);
 #pragma unroll
             for (int i = 0; i < U; ++i) {
                 const int n = n0 + i * rg_n;
@@ -537,49 +574,103 @@ __global__ void __launch_bounds__(256) mamba2_single_kernel(const Mamba2Args a, 
 }
 
 // ------------------------------------------------------------------------------------------------ gate and norm
-// out[t, c] = v[c] / sqrt(mean over c's part of v^2 + eps) * weight[c],  v = y silu(z); a block a row.  With `history` (steps
-// of single tokens) the block also moves its request's convolution history on by the row's x | B | C.
+// out[t, c] = v[c] / sqrt(mean over c's part of v^2 + eps) * weight[c],  v = y silu(z); block (row, part).  With `history` (steps
+// of single tokens) further blocks of a row move its request's convolution history on by the row's x | B | C.
 template <typename T>
 __global__ void __launch_bounds__(256) mamba2_norm_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ rows,
                                                           int stride, int z_at, const float* __restrict__ weight, float eps, int I,
-                                                          int parts, float* __restrict__ history, int xbc_at, int ch, int L,
+                                                          int parts, int vec, float* __restrict__ history, int xbc_at, int ch, int L,
                                                           const int* __restrict__ slot_ids, int num_slots, int* __restrict__ status) {
-    extern __shared__ __align__(16) float m2_smem[];
     __shared__ float red[33];
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.x, len = I / parts;
+    const int t = blockIdx.x, part = blockIdx.y, len = I / parts;
     const T* row = rows + (size_t)t * stride;
-    if (history && L > 1) {
+    if (part >= parts) {
+        const int c = (part - parts) * blockDim.x + threadIdx.x;
+        if (c >= ch) return;
         const int slot = zai_checked_slot(slot_ids[t], num_slots, status);
-        float* hist = history + (size_t)slot * (L - 1) * ch;
-        for (int c = threadIdx.x; c < ch; c += blockDim.x) {
-            float keep[M2_MAX_TAPS];
-            const float cur = to_float(row[xbc_at + c]);
-            for (int j = 1; j < L - 1; ++j) keep[j] = hist[(size_t)j * ch + c];
-            for (int j = 1; j < L - 1; ++j) hist[(size_t)(j - 1) * ch + c] = keep[j];
-            hist[(size_t)(L - 2) * ch + c] = cur;
-        }
+        float* hist = history + (size_t)slot * (L - 1) * ch + c;
+        float keep[M2_MAX_TAPS];
+#pragma unroll
+        for (int j = 1; j < M2_MAX_TAPS; ++j) keep[j] = j < L - 1 ? hist[(size_t)j * ch] : 0.f;
+        const float cur = to_float(row[xbc_at + c]);
+#pragma unroll
+        for (int j = 1; j < M2_MAX_TAPS; ++j)
+            if (j < L - 1) hist[(size_t)(j - 1) * ch] = keep[j];
+        hist[(size_t)(L - 2) * ch] = cur;
+        return;
     }
-    // warps take parts in turn when there are many, the whole block takes one part at a time when there are few
-    for (int c = threadIdx.x; c < I; c += blockDim.x) m2_smem[c] = y[(size_t)t * I + c] * m2_silu(to_float(row[z_at + c]));
-    __syncthreads();
-    if (parts >= 8) {
-        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-        for (int p = warp; p < parts; p += nw) {
-            float q = 0.f;
-            for (int c = lane; c < len; c += 32) q += m2_smem[p * len + c] * m2_smem[p * len + c];
-            const float inv = rsqrtf(warp_sum(q) / (float)len + eps);
-            for (int c = p * len + lane; c < (p + 1) * len; c += 32) out[(size_t)t * I + c] = from_float<T>(m2_smem[c] * inv * weight[c]);
+    const float* yp = y + (size_t)t * I + part * len;
+    const T* zp = row + z_at + part * len;
+    const float* wp = weight + part * len;
+    T* op = out + (size_t)t * I + part * len;
+    float q = 0.f;
+    if (vec) {                                   // eight values a thread and step; the first two steps' stay in registers
+        float v[2][8];
+        auto load8 = [&](int c, float (&d)[8]) {
+            const float4 a = *reinterpret_cast<const float4*>(yp + c), b = *reinterpret_cast<const float4*>(yp + c + 4);
+            const float yv[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+            float zv[8];
+            if constexpr (sizeof(T) == 2) {
+                const uint4 u = *reinterpret_cast<const uint4*>(zp + c);
+                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 f = __bfloat1622float2(h[i]);
+                    zv[2 * i] = f.x; zv[2 * i + 1] = f.y;
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) zv[i] = to_float(zp[c + i]);
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) d[i] = yv[i] * m2_silu(zv[i]);
+        };
+        auto store8 = [&](int c, const float (&d)[8], float inv) {
+            const float4 a = *reinterpret_cast<const float4*>(wp + c), b = *reinterpret_cast<const float4*>(wp + c + 4);
+            const float w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+            if constexpr (sizeof(T) == 2) {
+                uint32_t u[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) u[i] = pack_bf16(d[2 * i] * inv * w[2 * i], d[2 * i + 1] * inv * w[2 * i + 1]);
+                *reinterpret_cast<uint4*>(op + c) = make_uint4(u[0], u[1], u[2], u[3]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) op[c + i] = from_float<T>(d[i] * inv * w[i]);
+            }
+        };
+        const int step = blockDim.x * 8, c0 = threadIdx.x * 8;
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (c0 + k * step < len) {
+                load8(c0 + k * step, v[k]);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) q += v[k][i] * v[k][i];
+            }
+        for (int c = c0 + 2 * step; c < len; c += step) {
+            float d[8];
+            load8(c, d);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) q += d[i] * d[i];
+        }
+        const float inv = rsqrtf(block_sum(q, red) / (float)len + eps);
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (c0 + k * step < len) store8(c0 + k * step, v[k], inv);
+        for (int c = c0 + 2 * step; c < len; c += step) {
+            float d[8];
+            load8(c, d);
+            store8(c, d, inv);
         }
         return;
     }
-    for (int p = 0; p < parts; ++p) {
-        float q = 0.f;
-        for (int c = threadIdx.x; c < len; c += blockDim.x) q += m2_smem[p * len + c] * m2_smem[p * len + c];
-        const float inv = rsqrtf(block_sum(q, red) / (float)len + eps);
-        for (int c = p * len + threadIdx.x; c < (p + 1) * len; c += blockDim.x) out[(size_t)t * I + c] = from_float<T>(m2_smem[c] * inv * weight[c]);
+    for (int c = threadIdx.x; c < len; c += blockDim.x) {
+        const float v = yp[c] * m2_silu(to_float(zp[c]));
+        q += v * v;
     }
+    const float inv = rsqrtf(block_sum(q, red) / (float)len + eps);
+    for (int c = threadIdx.x; c < len; c += blockDim.x) op[c] = from_float<T>(yp[c] * m2_silu(to_float(zp[c])) * inv * wp[c]);
 }
 
 // ------------------------------------------------------------------------------------------------ launchers
@@ -636,7 +727,7 @@ static int m2_chunked(const Mamba2Args& a, float* ends, float* last, int max_chu
         if (e != cudaSuccess) return (int)e;
     }
     const dim3 grid(max_chunks, a.H, (a.V + VT - 1) / VT);
-    int rc = launch_pdl(mamba2_chunk_state_kernel<VT>, grid, dim3(128), m2_state_smem(a.N, VT), stream, a, ends, last);
+    int rc = launch_pdl(mamba2_chunk_state_kernel<VT>, grid, dim3(256), m2_state_smem(a.N, VT), stream, a, ends, last);
     if (rc) return rc;
     const size_t total = (size_t)a.H * a.N * a.V;
     if (((size_t)a.N * a.V) % 4 == 0)
@@ -644,7 +735,7 @@ static int m2_chunked(const Mamba2Args& a, float* ends, float* last, int max_chu
     else
         rc = launch_pdl(mamba2_state_pass_kernel<1>, dim3((unsigned)((total + 127) / 128), a.n_seqs), dim3(128), 0, stream, a, ends, (const float*)last);
     if (rc) return rc;
-    return launch_pdl(mamba2_chunk_out_kernel<VT>, grid, dim3(128), m2_out_smem(a.N, VT), stream, a, (const float*)ends);
+    return launch_pdl(mamba2_chunk_out_kernel<VT>, grid, dim3(256), m2_out_smem(a.N, VT), stream, a, (const float*)ends);
 }
 
 // The same over every span of min_rows rows or more, bfloat16, in chunks on the tensor cores.  ends [max_chunks, H, N, V] and
@@ -687,16 +778,15 @@ ZAI_API int zai_mamba2_norm(void* out, const float* y, const void* rows, int str
                             int N, int I, int parts, float* history, int xbc_at, int ch, int L, const int* slot_ids, int num_slots,
                             int* status, cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
-    if (I < 1 || parts < 1 || I % parts || I > 48 * 1024 || L > M2_MAX_TAPS) return ZAI_BAD_SIZE;
-    const size_t smem = (size_t)I * sizeof(float);
-    static unsigned long long done[2] = {0, 0};
-    if (dtype != ZAI_F32 && dtype != ZAI_BF16) return ZAI_BAD_DTYPE;
-    if (zai_first_on_device(&done[dtype])) {
-        cudaError_t e;
-        if (dtype == ZAI_F32) e = cudaFuncSetAttribute(mamba2_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 192 * 1024);
-        else e = cudaFuncSetAttribute(mamba2_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 192 * 1024);
-        if (e != cudaSuccess) return (int)e;
-    }
-    ZAI_DISPATCH(dtype, return launch_pdl(mamba2_norm_kernel<T>, dim3(N), dim3(256), smem, stream, (T*)out, y, (const T*)rows, stride, z_at,
-                                          weight, eps, I, parts, history, xbc_at, ch, L, slot_ids, num_slots, status));
+    if (I < 1 || parts < 1 || I % parts || L > M2_MAX_TAPS) return ZAI_BAD_SIZE;
+    const int len = I / parts;
+    const int vec = len % 8 == 0 && stride % 8 == 0 && z_at % 8 == 0
+                    && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(weight)) & 15) == 0;
+    int threads = ((vec ? len / 8 : len) + 31) / 32 * 32;
+    threads = threads > 256 ? 256 : threads;
+    const int moving = (history && L > 1) ? (ch + threads - 1) / threads : 0;
+    if (parts + moving > 65535) return ZAI_BAD_SIZE;
+    ZAI_DISPATCH(dtype, return launch_pdl(mamba2_norm_kernel<T>, dim3(N, parts + moving), dim3(threads), 0, stream, (T*)out, y,
+                                          (const T*)rows, stride, z_at, weight, eps, I, parts, vec, history, xbc_at, ch, L, slot_ids,
+                                          num_slots, status));
 }

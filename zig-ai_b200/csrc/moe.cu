@@ -16,18 +16,22 @@
 //     the tile height TM (padding rows hold whatever was there: a row's result never depends on another row), and the
 //     expert of every tile;
 //   * two grouped products over that layout (gate|up with the activation as epilogue, then down): a block owns a
-//     tile of TM rows x 64 output columns of one expert; bfloat16 on the tensor cores (mma.sync m16n8k16, cp.async
-//     ring of three stages), any other case by 32-bit multiply-adds.  Steps with many rows an expert gather with a
+//     tile of TM rows x 32 or 64 output columns of one expert; bfloat16 on the tensor cores (mma.sync m16n8k16, cp.async
+//     ring), any other case by 32-bit multiply-adds.  Steps with many rows an expert gather with a
 //     tile height of 128 and run both products in the grouped mode of the tcgen05 kernel (gemm_tc.cu) instead;
 //   * combine: a row's `top` results summed in 32-bit in the order of the choice and rounded once.
 // A row's result depends on the row alone: on which tile it lands, what else the tile holds and in which order the
 // counter was taken changes nothing, since every output element is a sum over k in a fixed order.
 #include "mma_helpers.cuh"
 
-#define MOE_TN 64          // output columns of a block
-#define MOE_TK 32          // k per stage
-#define MOE_ST (MOE_TK + 8)
-#define MOE_STAGES 3
+#define MOE_PLAIN_TN 64    // output columns of a block of the plain kernel
+#define MOE_PLAIN_TK 32    // k per stage of the plain kernel
+// Tiles of the tensor-core kernel by the tile height TM: output columns TN and warps of a block, k per stage, stages.  With few
+// rows a block mostly brings its weights in, one pass, so what it keeps in flight is what hides the way to memory.
+template <int TM> struct MoeTile {
+    static constexpr int TN = TM == 16 ? 32 : 64, WARPS = TM == 16 ? 2 : 4, TK = 64, ST = TK + 8, STAGES = TM == 16 ? 10 : 4;
+    static constexpr size_t BYTES = (size_t)STAGES * (TM + TN) * ST * 2;
+};
 
 // Eight neighbouring values as 32-bit numbers by 16-byte accesses (the caller has checked the alignment).
 __device__ __forceinline__ void moe_load8(float (&v)[8], const bf16* p) {
@@ -61,40 +65,55 @@ __device__ __forceinline__ bool moe_rows_aligned(const T* p, size_t stride, int 
 
 // ------------------------------------------------------------------------------------------------ route
 enum { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_LOGITS = 2 };          // what the scores are
-template <typename T>
-__global__ void __launch_bounds__(128) moe_route_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ rank,
+// ROWS rows a block (their values are read once per expert row of the router for all of them); a row's sums have the same order
+// whatever ROWS and the number of warps are.
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(512) moe_route_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ rank,
                                                         int* __restrict__ counts, const T* __restrict__ x, int x_stride,
-                                                        const float* __restrict__ wr, int W, int E, int top, int renorm,
+                                                        const float* __restrict__ wr, int N, int W, int E, int top, int renorm,
                                                         int score, const float* __restrict__ bias, float* __restrict__ unit_gate) {
-    extern __shared__ float sc[];                        // [E] scores
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    extern __shared__ float sc_all[];                    // [ROWS][E] scores
+    const int tr = blockIdx.x * ROWS, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     pdl_trigger();
     pdl_wait();
-    const T* row = x + (size_t)t * x_stride;
     // (which of the two loops runs depends on the sizes and addresses alone, never on the other rows of the step)
     const bool vec = moe_rows_aligned(x, (size_t)x_stride, W) && (reinterpret_cast<uintptr_t>(wr) & 15) == 0;
-    for (int e = warp; e < E + (unit_gate ? 1 : 0); e += 4) {
+    for (int e = warp; e < E + (unit_gate ? 1 : 0); e += nw) {
         const float* w = wr + (size_t)e * W;
-        float acc = 0.f;
+        float acc[ROWS];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
         if (vec) {
+#pragma unroll 4
             for (int c = lane * 8; c < W; c += 256) {
                 float xv[8], wv[8];
-                moe_load8(xv, row + c);
                 moe_load8(wv, w + c);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) acc += xv[i] * wv[i];
+                for (int r = 0; r < ROWS; ++r) {
+                    moe_load8(xv, x + (size_t)min(tr + r, N - 1) * x_stride + c);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) acc[r] += xv[i] * wv[i];
+                }
             }
         } else {
-            for (int c = lane; c < W; c += 32) acc += to_float(row[c]) * w[c];
+            for (int c = lane; c < W; c += 32) {
+                const float wv = w[c];
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) acc[r] += to_float(x[(size_t)min(tr + r, N - 1) * x_stride + c]) * wv;
+            }
         }
-        acc = warp_sum(acc);
-        if (lane == 0) {
-            if (e == E) unit_gate[t] = 1.f / (1.f + expf(-acc));         // (the row behind the router's: the unit beside the experts)
-            else sc[e] = score == MOE_SIGMOID ? 1.f / (1.f + expf(-acc)) : bias ? acc + bias[e] : acc;
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const float z = warp_sum(acc[r]);
+            if (lane != 0 || tr + r >= N) continue;
+            if (e == E) unit_gate[tr + r] = 1.f / (1.f + expf(-z));      // (the row behind the router's: the unit beside the experts)
+            else sc_all[r * E + e] = score == MOE_SIGMOID ? 1.f / (1.f + expf(-z)) : bias ? z + bias[e] : z;
         }
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int t = tr + warp;
+    if (warp >= ROWS || t >= N) return;
+    float* sc = sc_all + warp * E;
     if (score == MOE_SOFTMAX) {                          // scores = softmax of the logits over all experts, in a fixed order
         float top_z = -INFINITY;
         for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, sc[e]);
@@ -216,24 +235,28 @@ struct MoeAct {
     }
 };
 
-// The weight row that row r (0..63) of a block's tile of weights holds, or -1.  Plain: output column n0 + r.  Gated:
+// The weight row that row r (0..TN - 1) of a block's tile of weights holds, or -1.  Plain: output column n0 + r.  Gated:
 // groups of eight rows alternate between the gate and the up rows of the same eight features.
+template <int TN>
 __device__ __forceinline__ int moe_weight_row(int r, int col_block, int n_out, int gated) {
     if (!gated) {
-        const int n = col_block * MOE_TN + r;
+        const int n = col_block * TN + r;
         return n < n_out ? n : -1;
     }
-    const int f = col_block * (MOE_TN / 2) + (r >> 4) * 8 + (r & 7);
+    const int f = col_block * (TN / 2) + (r >> 4) * 8 + (r & 7);
     return f < n_out ? ((r >> 3) & 1) * n_out + f : -1;
 }
 
 template <int TM, typename TO>
-__global__ void __launch_bounds__(128) moe_gemm_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ xs,
+__global__ void __launch_bounds__(MoeTile<TM>::WARPS * 32) moe_gemm_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ xs,
                                                            const bf16* __restrict__ w, const int* __restrict__ tile_expert,
                                                            int K, int n_out, int gated, const MoeAct act) {
-    constexpr int WM = TM / 16, WN = 4 / WM, NT = 8 / WN;            // warps along rows and columns; 8-column tiles a warp
-    __shared__ __align__(16) bf16 sa[MOE_STAGES][TM][MOE_ST];
-    __shared__ __align__(16) bf16 sb[MOE_STAGES][MOE_TN][MOE_ST];
+    constexpr int MOE_TN = MoeTile<TM>::TN, THREADS = MoeTile<TM>::WARPS * 32;
+    constexpr int WM = TM / 16, WN = MoeTile<TM>::WARPS / WM, NT = MOE_TN / 8 / WN;   // warps along rows and columns; 8-column tiles a warp
+    constexpr int MOE_TK = MoeTile<TM>::TK, MOE_ST = MoeTile<TM>::ST, MOE_STAGES = MoeTile<TM>::STAGES;
+    extern __shared__ __align__(16) unsigned char moe_raw[];
+    bf16 (*sa)[TM][MOE_ST] = reinterpret_cast<bf16 (*)[TM][MOE_ST]>(moe_raw);
+    bf16 (*sb)[MOE_TN][MOE_ST] = reinterpret_cast<bf16 (*)[MOE_TN][MOE_ST]>(moe_raw + (size_t)MOE_STAGES * TM * MOE_ST * 2);
     pdl_trigger();
     pdl_wait();
     const int e = tile_expert[blockIdx.x];
@@ -245,14 +268,14 @@ __global__ void __launch_bounds__(128) moe_gemm_mma_kernel(TO* __restrict__ out,
     const int n_k = (K + MOE_TK - 1) / MOE_TK;
     auto load = [&](int kt, int buf) {
         const int k0 = kt * MOE_TK;
-        for (int i = tid; i < TM * (MOE_TK / 8); i += 128) {
+        for (int i = tid; i < TM * (MOE_TK / 8); i += THREADS) {
             const int r = i / (MOE_TK / 8), c = (i % (MOE_TK / 8)) * 8;
             const bool ok = k0 + c < K;
             cp_async16(&sa[buf][r][c], xs + (row0 + r) * K + (ok ? k0 + c : 0), ok);
         }
-        for (int i = tid; i < MOE_TN * (MOE_TK / 8); i += 128) {
+        for (int i = tid; i < MOE_TN * (MOE_TK / 8); i += THREADS) {
             const int r = i / (MOE_TK / 8), c = (i % (MOE_TK / 8)) * 8;
-            const int wr = moe_weight_row(r, blockIdx.y, n_out, gated);
+            const int wr = moe_weight_row<MOE_TN>(r, blockIdx.y, n_out, gated);
             const bool ok = wr >= 0 && k0 + c < K;
             cp_async16(&sb[buf][r][c], wexp + (ok ? (size_t)wr * K + k0 + c : 0), ok);
         }
@@ -320,8 +343,8 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(128) moe_gemm_plain_kernel(TO* __restrict__ out, const T* __restrict__ xs, const T* __restrict__ w,
                                                              const int* __restrict__ tile_expert, int K, int n_out, int gated,
                                                              const MoeAct act) {
-    __shared__ float sa[16][MOE_TK + 1];
-    __shared__ float sb[MOE_TN][MOE_TK + 1];
+    __shared__ float sa[16][MOE_PLAIN_TK + 1];
+    __shared__ float sb[MOE_PLAIN_TN][MOE_PLAIN_TK + 1];
     pdl_trigger();
     pdl_wait();
     const int e = tile_expert[blockIdx.x];
@@ -332,20 +355,20 @@ __global__ void __launch_bounds__(128) moe_gemm_plain_kernel(TO* __restrict__ ou
     float acc[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] = 0.f;
-    for (int k0 = 0; k0 < K; k0 += MOE_TK) {
+    for (int k0 = 0; k0 < K; k0 += MOE_PLAIN_TK) {
         __syncthreads();
-        for (int i = tid; i < 16 * MOE_TK; i += 128) {
-            const int rr = i / MOE_TK, kk = i % MOE_TK;
+        for (int i = tid; i < 16 * MOE_PLAIN_TK; i += 128) {
+            const int rr = i / MOE_PLAIN_TK, kk = i % MOE_PLAIN_TK;
             sa[rr][kk] = k0 + kk < K ? to_float(xs[(row0 + rr) * K + k0 + kk]) : 0.f;
         }
-        for (int i = tid; i < MOE_TN * MOE_TK; i += 128) {
-            const int rr = i / MOE_TK, kk = i % MOE_TK;
-            const int wr = moe_weight_row(rr, blockIdx.y, n_out, gated);
+        for (int i = tid; i < MOE_PLAIN_TN * MOE_PLAIN_TK; i += 128) {
+            const int rr = i / MOE_PLAIN_TK, kk = i % MOE_PLAIN_TK;
+            const int wr = moe_weight_row<MOE_PLAIN_TN>(rr, blockIdx.y, n_out, gated);
             sb[rr][kk] = (wr >= 0 && k0 + kk < K) ? to_float(wexp[(size_t)wr * K + k0 + kk]) : 0.f;
         }
         __syncthreads();
 #pragma unroll 4
-        for (int kk = 0; kk < MOE_TK; ++kk) {
+        for (int kk = 0; kk < MOE_PLAIN_TK; ++kk) {
             const float a = sa[r][kk];
 #pragma unroll
             for (int j = 0; j < 8; ++j) acc[j] = fmaf(a, sb[c8 + 8 * j][kk], acc[j]);
@@ -355,14 +378,14 @@ __global__ void __launch_bounds__(128) moe_gemm_plain_kernel(TO* __restrict__ ou
     if (gated) {
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
-            const int f = blockIdx.y * (MOE_TN / 2) + (j / 2) * 8 + c8;
+            const int f = blockIdx.y * (MOE_PLAIN_TN / 2) + (j / 2) * 8 + c8;
             if (f < n_out) moe_store<TO>(out + (row0 + r) * n_out + f, act(acc[j], acc[j + 1]));
         }
         return;
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-        const int n = blockIdx.y * MOE_TN + c8 + 8 * j;
+        const int n = blockIdx.y * MOE_PLAIN_TN + c8 + 8 * j;
         if (n < n_out) moe_store<TO>(out + (row0 + r) * n_out + n, act.plain(acc[j]));
     }
 }
@@ -418,8 +441,14 @@ ZAI_API int zai_moe_route(int* ids, float* wts, int* rank, int* counts, const vo
     if (E < 1 || top < 1 || top > E || top > 32 || E > 8192 || W < 1 || score < MOE_SIGMOID || score > MOE_LOGITS || (bias && score == MOE_SIGMOID)) return ZAI_BAD_SIZE;
     cudaError_t rc = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int), stream);
     if (rc != cudaSuccess) return (int)rc;
-    ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T>, dim3(N), dim3(128), (size_t)E * sizeof(float), stream, ids, wts, rank,
-                                          counts, (const T*)x, x_stride, wr, W, E, top, renorm, score, bias, unit_gate));
+    const int rows = E + (unit_gate ? 1 : 0);
+    if (N >= 512 && E <= 2048) {
+        ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 4>, dim3((N + 3) / 4), dim3(rows <= 4 ? 128 : 256), (size_t)4 * E * sizeof(float),
+                                              stream, ids, wts, rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate));
+    }
+    const int warps = rows < 4 ? 4 : rows > 16 ? 16 : rows;
+    ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 1>, dim3(N), dim3(warps * 32), (size_t)E * sizeof(float), stream, ids, wts,
+                                          rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate));
 }
 
 // The most tiles of TM rows that N x top choices over E experts can take.
@@ -441,6 +470,17 @@ ZAI_API int zai_moe_gather(void* xs, int* dest, int* tile_expert, const void* x,
                                           max_tiles, scale_input));
 }
 
+template <int TM, typename TO>
+static int moe_launch_mma(dim3 grid, TO* out, const bf16* xs, const bf16* w, const int* tile_expert, int K, int n_out, int gated,
+                          const MoeAct& act, cudaStream_t stream) {
+    static unsigned long long done = 0;
+    if (zai_first_on_device(&done)) {
+        cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel<TM, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MoeTile<TM>::BYTES);
+        if (e != cudaSuccess) return (int)e;
+    }
+    return launch_pdl(moe_gemm_mma_kernel<TM, TO>, grid, dim3(MoeTile<TM>::WARPS * 32), MoeTile<TM>::BYTES, stream, out, xs, w, tile_expert, K, n_out, gated, act);
+}
+
 // out [max_tiles * TM, n_out] (32-bit if out_f32, else `dtype`) = xs [max_tiles * TM, K] . w[expert of the tile]^T;
 // w [E, n_out, K], or with kind 1 or 2 [E, 2 n_out, K] and out = silu(gate) * up (kind 1) or the bounded gated activation with
 // `limit` and `alpha` (kind 2); kind 3: the square of relu on the plain products.  TM 16 or 64 (the gather's).
@@ -451,12 +491,12 @@ ZAI_API int zai_moe_gemm(void* out, int out_f32, const void* xs, const void* w, 
     const MoeAct act = {kind, limit, alpha};
     const int gated = kind == 1 || kind == 2;
     if (K < 1 || n_out < 1 || (TM != 16 && TM != 64)) return ZAI_BAD_SIZE;
-    const int cols = gated ? MOE_TN / 2 : MOE_TN;
+    const bool mma = dtype == ZAI_BF16 && K % 8 == 0;
+    const int tn = mma ? (TM == 16 ? MoeTile<16>::TN : MoeTile<64>::TN) : MOE_PLAIN_TN, cols = gated ? tn / 2 : tn;
     const dim3 grid(max_tiles, (n_out + cols - 1) / cols);
     if (grid.y > 65535) return ZAI_BAD_SIZE;
-    if (dtype == ZAI_BF16 && K % 8 == 0) {
-#define MOE_GO(TMV, TOV) return launch_pdl(moe_gemm_mma_kernel<TMV, TOV>, grid, dim3(128), 0, stream, (TOV*)out, (const bf16*)xs, \
-                                           (const bf16*)w, tile_expert, K, n_out, gated, act)
+    if (mma) {
+#define MOE_GO(TMV, TOV) return moe_launch_mma<TMV, TOV>(grid, (TOV*)out, (const bf16*)xs, (const bf16*)w, tile_expert, K, n_out, gated, act, stream)
         if (TM == 16) { if (out_f32) MOE_GO(16, float); else MOE_GO(16, bf16); }
         if (out_f32) MOE_GO(64, float); else MOE_GO(64, bf16);
 #undef MOE_GO
