@@ -216,7 +216,7 @@ def cancellation(m, w, h):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,D,V,window", [(4, 2, 32, 64, 24), (2, 1, 16, 24, 5), (3, 3, 8, 40, 70), (4, 1, 64, 128, 33), (2, 2, 20, 40, 1),
+@pytest.mark.parametrize("H,G,D,V,window", [(6, 2, 32, 64, 24), (2, 1, 16, 24, 5), (3, 3, 8, 40, 70), (4, 1, 64, 128, 33), (2, 2, 20, 40, 1),
                                             (6, 2, 24, 16, 1000)])
 def test_differential_attention_with_planted_keys(dtype, H, G, D, V, window):
     """The part over cached pages against the formula, with one key made to match the last row's query in one of the two maps: just
