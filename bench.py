@@ -1098,17 +1098,18 @@ def sogenex_kernel_rooflines(width, hbm_peak, flops_peak):
         maps = qkv[:, :2 * Ha * V].reshape(N, Ha, 2, 2, D)
         maps[:, :, 0, 1] = 0
         maps[:, :, 1, 0] = 0
+        paired = qkv[:, Ha * V:].contiguous()               # (a step of single tokens: from the projection's rows)
 
-        def plain(view, qkv, H, G, Dh):
+        def plain(view, qkv, H, G, Dh, q_map=0):
             if N == B:
-                return lambda: ops.decode_attention_fused(qkv, None, None, 0.0, 0, 1.0, step, view, H, G, Dh, 0.125, 1024)
+                return lambda: ops.decode_attention_fused(qkv, None, None, 0.0, 0, 1.0, step, view, H, G, Dh, 0.125, 1024, q_map=q_map)
             q = qkv[:, :H * Dh].contiguous()
             return lambda: ops.paged_attention(q, step, view, H, G, Dh, 0.125, 1024)
-        two = plain(view, qkv, 2 * Ha, Ga, V)
+        two, one = plain(view, paired if N == B else qkv, 2 * Ha, Ga, V, D), plain(view, qkv, 2 * Ha, Ga, V)
         fl, by = 2.0 * pairs * 2 * Ha * (D + V), cached * Ga * 2 * V * 2 + N * Ha * (2 * D + V) * 2
         rows.append(("differential attention: two maps, their difference normed", point,
                      timed(lambda: ops.attention_difference(two(), Ha, V, V, 0.5, 0.5, 1e-6)), fl, by))
-        rows.append(("windowed attention, heads of 128 (LFM2's kernels)", point, timed(two), 2.0 * pairs * 2 * Ha * 2 * V,
+        rows.append(("windowed attention, heads of 128 (LFM2's kernels)", point, timed(one), 2.0 * pairs * 2 * Ha * 2 * V,
                      cached * Ga * 2 * V * 2 + N * Ha * 4 * V * 2))
         view64 = CacheView(0, rnd(n_pages, 2, 2 * Ga, ps, D, s=0.5), step.block_tables[0], ps)
         qkv64 = rnd(N, (2 * Ha + 4 * Ga) * D)

@@ -166,9 +166,14 @@ def _page_rows(step, cache):
 
 
 def qk_norm_rope(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_heads, head_dim,
-                 has_kv=True, write=True, return_k=False):
+                 has_kv=True, write=True, return_k=False, q_map=0):
     N = qkv.shape[0]
     D = head_dim
+    if q_map:                            # heads / 2 query heads of two maps each: a query head per map, zeros in the other's place
+        pairs = qkv[:, :heads // 2 * D].reshape(N, heads // 2, 1, D).repeat(1, 1, 2, 1)
+        pairs[:, :, 0, q_map:] = 0
+        pairs[:, :, 1, :q_map] = 0
+        qkv = torch.cat([pairs.reshape(N, heads * D), qkv[:, heads // 2 * D:]], dim=1)
     q = _f(qkv[:, :heads * D]).reshape(N, heads, D)
     if q_w is not None:
         q = _rms(q, q_w, eps)

@@ -569,6 +569,7 @@ struct FusedDecodeArgs {
     const int* block_table;
     const int* positions;
     float eps, scale_log2;
+    int q_map;                 // > 0: the projection holds pairs of maps (query_head)
     int qkv_cols, rot, table_width, page_size, Hq, Hkv, window, write_kv;
     int num_pages;             // pages in `pages`: a table entry outside is read as page 0 and raises the status word
     int* status;
@@ -620,14 +621,18 @@ __global__ void __launch_bounds__(NTHREADS) decode_fused_kernel(const FusedDecod
         cp_async_commit();
         // meanwhile: the group's queries, and the new key and value
         const bf16* row = a.qkv + (size_t)b * a.qkv_cols;
+        const int q_rows = a.q_map > 0 ? Hq / 2 : Hq;           // query heads that the projection's rows hold
         const float2* cs = a.rot ? a.cs_table + (size_t)b * (a.rot >> 1) : nullptr;
         for (int r = warp; r < 16; r += 4) {
-            if (r < G) norm_rotate_row<D>(row + (size_t)(hk * G + r) * D, a.q_gamma, a.eps, cs, a.rot, tmp + warp * D, sq + r * ST, lane);
+            if (r < G) {
+                const QueryHead qh = query_head(hk * G + r, D, a.q_map);
+                norm_rotate_row<D>(row + (size_t)qh.source * D, a.q_gamma, a.eps, cs, a.rot, tmp + warp * D, sq + r * ST, lane, qh.keep0, qh.keep1);
+            }
             else for (int d = lane; d < D; d += 32) sq[r * ST + d] = __float2bfloat16_rn(0.f);
         }
         if (has_new && warp == 0) {
-            norm_rotate_row<D>(row + (size_t)(Hq + hk) * D, a.k_gamma, a.eps, cs, a.rot, tmp, knew, lane);
-            const bf16* vraw = row + (size_t)(Hq + Hkv + hk) * D;
+            norm_rotate_row<D>(row + (size_t)(q_rows + hk) * D, a.k_gamma, a.eps, cs, a.rot, tmp, knew, lane);
+            const bf16* vraw = row + (size_t)(q_rows + Hkv + hk) * D;
             int page, off;
             if (page_shift >= 0) { page = table.page(pos >> page_shift); off = pos & (page_size - 1); }
             else { page = table.page(pos / page_size); off = pos % page_size; }
@@ -961,21 +966,23 @@ ZAI_API int zai_decode_attention_mma(void* out, float* part_o, float* part_ml, c
 }
 
 // The decode step's attention from the raw qkv rows: see decode_fused_kernel.  `tickets` holds
-// B * Hkv zeros (and again after the call).
+// B * Hkv zeros (and again after the call).  q_map > 0: the rows hold Hq / 2 query heads, each two maps of q_map and D - q_map
+// values, which count as two query heads with zeros in the other map's place (no norm, no rotation).
 ZAI_API int zai_decode_attention_fused(void* out, float* part_o, float* part_ml, int* tickets, const void* qkv,
                                        int qkv_cols, const float* q_gamma, const float* k_gamma, float eps,
                                        const float2* cs_table, int rot, void* pages, const int* block_table,
                                        int table_width, const int* positions, int B, int n_chunks, int page_size,
                                        int Hq, int Hkv, int D, float scale, int window, int write_kv, int chunk_keys,
-                                       int num_pages, int* status, cudaStream_t stream) {
+                                       int num_pages, int* status, int q_map, cudaStream_t stream) {
     if (B <= 0) return ZAI_OK;
+    if (q_map < 0 || q_map > D || (q_map && ((Hq & 1) || rot || q_gamma))) return ZAI_BAD_SIZE;
     if (chunk_keys < TILE || chunk_keys % TILE) return ZAI_BAD_SIZE;
     if (n_chunks < 1 || Hkv < 1 || Hkv > 65535 || B > 65535 || Hq % Hkv != 0 || Hq / Hkv > 16 || rot < 0 || rot > D || (rot & 1))
         return ZAI_BAD_SIZE;
     FusedDecodeArgs a;
     a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.tickets = tickets; a.qkv = (const bf16*)qkv;
     a.q_gamma = q_gamma; a.k_gamma = k_gamma; a.cs_table = cs_table; a.pages = (bf16*)pages; a.block_table = block_table;
-    a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot;
+    a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot; a.q_map = q_map;
     a.table_width = table_width; a.page_size = page_size; a.Hq = Hq; a.Hkv = Hkv; a.window = window; a.write_kv = write_kv; a.chunk_keys = chunk_keys;
     a.num_pages = num_pages; a.status = status;
 #define X(d) if (D == d) return launch_decode_fused<d>(a, B, n_chunks, stream);

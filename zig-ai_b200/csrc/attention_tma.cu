@@ -95,6 +95,7 @@ struct TmaDecodeArgs {
     const int* block_table;
     const int* positions;
     float eps, scale_log2;
+    int q_map;                 // > 0: the projection holds pairs of maps (query_head)
     int qkv_cols, rot, table_width, page_size, page_shift, Hq, Hkv, window, write_kv, chunk_keys, stages;
     int chunk_fastest;         // the grid is (chunks, Hkv, B) if set, else (Hkv, B, chunks)
 };
@@ -205,15 +206,19 @@ __global__ void __maxnreg__(128) decode_tma_kernel(const __grid_constant__ CUten
         } else {
             // ---- consumers: first the group's queries, and the new key and value
             const bf16* row = a.qkv + (size_t)b * a.qkv_cols;
+            const int q_rows = a.q_map > 0 ? Hq / 2 : Hq;           // query heads that the projection's rows hold
             const float2* cs = a.rot ? a.cs_table + (size_t)b * (a.rot >> 1) : nullptr;
             // the rows to prepare (the group's G queries, then the new key) go round the warps
             for (int r = cw; r < 16; r += TT_CONSUMERS) {
-                if (r < G) norm_rotate_row<D>(row + (size_t)(hk * G + r) * D, a.q_gamma, a.eps, cs, a.rot, tmp + cw * D, sq + r * ST, lane);
+                if (r < G) {
+                    const QueryHead qh = query_head(hk * G + r, D, a.q_map);
+                    norm_rotate_row<D>(row + (size_t)qh.source * D, a.q_gamma, a.eps, cs, a.rot, tmp + cw * D, sq + r * ST, lane, qh.keep0, qh.keep1);
+                }
                 else for (int d = lane; d < D; d += 32) sq[r * ST + d] = __float2bfloat16_rn(0.f);
             }
             if (has_new && cw == G % TT_CONSUMERS) {
-                norm_rotate_row<D>(row + (size_t)(Hq + hk) * D, a.k_gamma, a.eps, cs, a.rot, tmp + cw * D, knew, lane);
-                const bf16* vraw = row + (size_t)(Hq + Hkv + hk) * D;
+                norm_rotate_row<D>(row + (size_t)(q_rows + hk) * D, a.k_gamma, a.eps, cs, a.rot, tmp + cw * D, knew, lane);
+                const bf16* vraw = row + (size_t)(q_rows + Hkv + hk) * D;
                 const int page = zai_checked_page(table, a.table_width, pos < 0 ? -1 : pos >> a.page_shift, a.num_pages,
                                                   lane == 0 ? a.status : nullptr);
                 const int off = pos & (ps - 1);
@@ -447,8 +452,9 @@ ZAI_API int zai_decode_attention_tma(void* out, float* part_o, float* part_ml, i
                                      const float2* cs_table, int rot, void* pages, int num_pages, const int* block_table,
                                      int table_width, const int* positions, int B, int n_chunks, int page_size, int Hq,
                                      int Hkv, int D, float scale, int window, int write_kv, int chunk_keys,
-                                     cudaStream_t stream) {
+                                     int q_map, cudaStream_t stream) {
     if (B <= 0) return ZAI_OK;
+    if (q_map < 0 || q_map > D || (q_map && ((Hq & 1) || rot || q_gamma))) return ZAI_BAD_SIZE;
     if (!zai_decode_attention_tma_supports(D, Hq, Hkv, page_size)) return ZAI_BAD_SIZE;
     if (chunk_keys < TT_TILE || chunk_keys % TT_TILE || n_chunks < 1 || Hkv > 65535 || B > 65535 || n_chunks > 65535 || rot < 0 || rot > D || (rot & 1))
         return ZAI_BAD_SIZE;
@@ -465,7 +471,7 @@ ZAI_API int zai_decode_attention_tma(void* out, float* part_o, float* part_ml, i
     TmaDecodeArgs a;
     a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.tickets = tickets; a.status = status; a.num_pages = num_pages; a.qkv = (const bf16*)qkv;
     a.q_gamma = q_gamma; a.k_gamma = k_gamma; a.cs_table = cs_table; a.pages = (bf16*)pages; a.block_table = block_table;
-    a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot;
+    a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot; a.q_map = q_map;
     a.table_width = table_width; a.page_size = page_size; a.Hq = Hq; a.Hkv = Hkv; a.window = window; a.write_kv = write_kv;
     a.chunk_keys = chunk_keys;
     a.page_shift = 0;

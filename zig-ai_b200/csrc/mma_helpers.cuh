@@ -44,10 +44,11 @@ __device__ __forceinline__ float fast_exp2(float x) {
 
 // one head row: RMSNorm (if gamma) and rotation of the first `rot` dims; `tmp` holds D floats.  The
 // row, the norm's weight and the rotation's cosines and sines are all asked for before the first
-// of them is used, so the three loads cost one trip to memory, not three.
+// of them is used, so the three loads cost one trip to memory, not three.  Values outside [keep0, keep1) count as zeros.
 template <int D>
 __device__ __forceinline__ void norm_rotate_row(const bf16* __restrict__ raw, const float* __restrict__ gamma, float eps,
-                                                const float2* __restrict__ cs, int rot, float* tmp, bf16* dst, int lane) {
+                                                const float2* __restrict__ cs, int rot, float* tmp, bf16* dst, int lane,
+                                                int keep0 = 0, int keep1 = D) {
     constexpr int PER = (D + 31) / 32;
     const int half = rot >> 1;
     float v[PER], gm[PER];
@@ -59,7 +60,7 @@ __device__ __forceinline__ void norm_rotate_row(const bf16* __restrict__ raw, co
         gm[i] = 1.f;
         c[i] = make_float2(1.f, 0.f);
         if (d < D) {
-            v[i] = __bfloat162float(raw[d]);
+            if (d >= keep0 && d < keep1) v[i] = __bfloat162float(raw[d]);
             if (gamma) gm[i] = gamma[d];
             if (d < rot) c[i] = cs[d < half ? d : d - half];
         }
@@ -93,4 +94,12 @@ __device__ __forceinline__ void norm_rotate_row(const bf16* __restrict__ raw, co
         }
     }
     __syncwarp();
+}
+
+// Where query head h of a projection row lies and what of it counts.  With q_map > 0 the row's query heads are pairs of maps:
+// heads 2 i and 2 i + 1 are both read from the i-th, and keep its values below q_map and from there on.
+struct QueryHead { int source, keep0, keep1; };
+__device__ __forceinline__ QueryHead query_head(int h, int D, int q_map) {
+    if (q_map <= 0) return {h, 0, D};
+    return (h & 1) ? QueryHead{h >> 1, q_map, D} : QueryHead{h >> 1, 0, q_map};
 }

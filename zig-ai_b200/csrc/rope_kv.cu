@@ -13,7 +13,7 @@
 // cosine are taken in 64-bit and rounded to 32-bit once per token and step (rope_table_kernel),
 // then shared by all heads and all layers with the same rotation.
 // One block per token; each warp takes heads in turn.
-#include "common.cuh"
+#include "mma_helpers.cuh"
 
 // table[t][i] = magnitude * (cos, sin) of positions[t] * inv_freq[i]
 __global__ void rope_table_kernel(float2* __restrict__ table, const int* __restrict__ positions,
@@ -34,7 +34,7 @@ __global__ void qk_norm_rope_kernel(const T* __restrict__ qkv, int qkv_cols, con
                                     int rot, const int* __restrict__ positions, const int* __restrict__ seq_idx,
                                     const int* __restrict__ block_table, int table_width, T* __restrict__ pages,
                                     int page_size, T* __restrict__ q_out, T* __restrict__ k_out, int Hq, int Hkv,
-                                    int D, int has_kv, int write, int num_pages, int* __restrict__ status) {
+                                    int D, int has_kv, int write, int num_pages, int* __restrict__ status, int q_map) {
     extern __shared__ float smem[];
     const int half = rot / 2;
     float* cs = smem;                       // [half] cos
@@ -62,7 +62,8 @@ __global__ void qk_norm_rope_kernel(const T* __restrict__ qkv, int qkv_cols, con
     const int n_heads = Hq + (has_kv ? 2 * Hkv : 0);
     const T* row = qkv + (size_t)t * qkv_cols;
     for (int h = warp; h < n_heads; h += nwarp) {
-        const T* x = row + (size_t)h * D;
+        const QueryHead qh = query_head(h, D, h < Hq ? q_map : 0);
+        const T* x = row + (size_t)(h < Hq ? qh.source : q_map > 0 ? h - Hq / 2 : h) * D;
         if (h >= Hq + Hkv) {                                  // a value head: copy into its page
             if (write) {
                 T* dst = pages + page_base + (((size_t)1 * Hkv + (h - Hq - Hkv)) * page_size + off) * D;
@@ -74,7 +75,7 @@ __global__ void qk_norm_rope_kernel(const T* __restrict__ qkv, int qkv_cols, con
         const float* gamma = is_q ? q_gamma : k_gamma;
         float ss = 0.f;
         for (int d = lane; d < D; d += 32) {
-            const float v = to_float(x[d]);
+            const float v = d >= qh.keep0 && d < qh.keep1 ? to_float(x[d]) : 0.f;
             buf[d] = v;
             ss += v * v;
         }
@@ -373,12 +374,15 @@ ZAI_API int zai_rope_table_scaled(float2* table, const int* positions, const dou
                       magnitude);
 }
 
+// q_map > 0: the rows hold Hq / 2 query heads, each two maps of q_map and D - q_map values; q_out has a query head per map with
+// zeros in the other map's place (no norm, no rotation).
 ZAI_API int zai_qk_norm_rope(const void* qkv, int qkv_cols, int dtype, const float* q_gamma, const float* k_gamma,
                              float eps, const float2* cs_table, int rot, const int* positions, const int* seq_idx,
                              const int* block_table, int table_width, void* pages, int page_size, void* q_out,
                              void* k_out, int N, int Hq, int Hkv, int D, int has_kv, int write, int num_pages,
-                             int* status, cudaStream_t stream) {
+                             int* status, int q_map, cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
+    if (q_map < 0 || q_map > D || (q_map && ((Hq & 1) || rot || q_gamma))) return ZAI_BAD_SIZE;
     if (rot < 0 || rot > D || (rot & 1) || D < 1) return ZAI_BAD_SIZE;
     // the vector kernel: bfloat16, the whole head rotated, 16-byte aligned rows and tables
     const uintptr_t all = reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(q_gamma) | reinterpret_cast<uintptr_t>(k_gamma) |
@@ -400,7 +404,7 @@ ZAI_API int zai_qk_norm_rope(const void* qkv, int qkv_cols, int dtype, const flo
     if (smem > 48 * 1024) return ZAI_BAD_SIZE;
     ZAI_DISPATCH(dtype, return launch_pdl(qk_norm_rope_kernel<T>, dim3(N), dim3(threads), smem, stream,
         (const T*)qkv, qkv_cols, q_gamma, k_gamma, eps, cs_table, rot, positions, seq_idx, block_table,
-        table_width, (T*)pages, page_size, (T*)q_out, (T*)k_out, Hq, Hkv, D, has_kv, write, num_pages, status));
+        table_width, (T*)pages, page_size, (T*)q_out, (T*)k_out, Hq, Hkv, D, has_kv, write, num_pages, status, q_map));
 }
 
 ZAI_API int zai_kv_write(const void* k, int k_stride, const void* v, int v_stride, int dtype, const int* positions,

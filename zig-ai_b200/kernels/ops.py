@@ -85,7 +85,7 @@ _SIGNATURES = {
         "zai_rope_table": [_P, _P, _P, _I, _I, _P],
         "zai_rope_table_scaled": [_P, _P, _P, _I, _I, ctypes.c_double, _P],
         "zai_qk_norm_rope": [_P, _I, _I, _P, _P, _F, _P, _I, _P, _P, _P, _I, _P, _I, _P, _P,
-                             _I, _I, _I, _I, _I, _I, _I, _P, _P],
+                             _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
         "zai_kv_write": [_P, _I, _P, _I, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
         "zai_value_norm_pad": [_P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P],
     },
@@ -103,7 +103,7 @@ _SIGNATURES = {
         "zai_decode_attention_mma_scored": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _P, _I, _P, _I,
                                             _P],
         "zai_decode_attention_fused": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I,
-                                       _F, _I, _I, _I, _I, _P, _P],
+                                       _F, _I, _I, _I, _I, _P, _I, _P],
         "zai_decode_chunk_keys": [],
         "zai_prefill_block_rows": [],
     },
@@ -136,7 +136,7 @@ _SIGNATURES = {
     "attention_tma": {
         "zai_decode_attention_tma_supports": [_I, _I, _I, _I],
         "zai_decode_attention_tma": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I,
-                                     _I, _F, _I, _I, _I, _P],
+                                     _I, _F, _I, _I, _I, _I, _P],
     },
     "attention_tc": {
         "zai_prefill_attention_tc_supports": [_I, _I, _I, _I],
@@ -870,8 +870,12 @@ def rope_table(step, rotary_dim: int, theta: float, device, scaling=None) -> tor
 
 @_timed("q/k norm, rotation, page write")
 def qk_norm_rope(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_heads, head_dim,
-                 has_kv=True, write=True, return_k=False):
+                 has_kv=True, write=True, return_k=False, q_map=0):
+    """q, k and v heads of projection rows: norm, rotation, page write.  `q_map` > 0: the rows hold heads / 2 query heads of two
+    maps each, which come out as a query head per map with zeros in the other map's place (no norm, no rotation)."""
     _cuda(qkv, q_w, k_w)
+    if qkv.shape[1] < ((heads // 2 if q_map else heads) + (2 * kv_heads if has_kv else 0)) * head_dim:
+        raise KernelError("qk_norm_rope: the rows do not hold the heads")
     N, cols = qkv.shape
     q = torch.empty((N, heads * head_dim), dtype=qkv.dtype, device=qkv.device)
     k_out = torch.empty((N, kv_heads * head_dim), dtype=qkv.dtype, device=qkv.device) if (return_k and has_kv) else None
@@ -885,7 +889,7 @@ def qk_norm_rope(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_h
         _ptr(step.positions), _ptr(step.seq_idx), _ptr(bt) if do_write else None,
         bt.shape[1] if do_write else 0, _ptr(pages) if do_write else None, cache.page_size, _ptr(q), _ptr(k_out),
         N, heads, kv_heads, head_dim, int(has_kv), int(do_write), pages.shape[0] if do_write else 0,
-        _status_ptr(qkv.device), _stream()), "qk_norm_rope")
+        _status_ptr(qkv.device), int(q_map), _stream()), "qk_norm_rope")
     return q, k_out
 
 
@@ -1048,12 +1052,14 @@ def fused_decode_attention_available(dtype, heads, kv_heads, head_dim) -> bool:
 
 @_timed("attention (with q/k norm, rotation, page write)")
 def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_heads, head_dim, scale,
-                           window=None, write=True):
+                           window=None, write=True, q_map=0):
     """A decode step's attention in one kernel, from the qkv projection's rows [B, (Hq + 2 Hkv) D]:
     q/k RMSNorm, rotation, the new key and value into their page, attention over the pages in chunks
-    of keys, and the combination of the chunks.  Every row of the step is one token."""
+    of keys, and the combination of the chunks.  Every row of the step is one token.  `q_map`: as in `qk_norm_rope`."""
     _cuda(qkv, q_w, k_w)
     B, cols = qkv.shape
+    if cols < ((heads // 2 if q_map else heads) + 2 * kv_heads) * head_dim:
+        raise KernelError("decode_attention_fused: the rows do not hold the heads")
     if B != step.n_tokens:
         raise KernelError(f"{B} rows for a step of {step.n_tokens} rows")
     dev = qkv.device
@@ -1080,13 +1086,13 @@ def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, h
             _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _status_ptr(dev), _ptr(qkv), cols, _ptr(q_w), _ptr(k_w),
             float(eps), _ptr(table), int(rotary_dim), _ptr(cache.pages), cache.pages.shape[0], _ptr(bt), bt.shape[1],
             _ptr(step.positions), B, n_chunks, cache.page_size, heads, kv_heads, head_dim, float(scale), int(window or 0),
-            int(bool(write)), chunk, _stream()), "decode_attention_tma")
+            int(bool(write)), chunk, int(q_map), _stream()), "decode_attention_tma")
         return out
     _check(_fn("attention_mma", "zai_decode_attention_fused")(
         _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _ptr(qkv), cols, _ptr(q_w), _ptr(k_w), float(eps),
         _ptr(table), int(rotary_dim), _ptr(cache.pages), _ptr(bt), bt.shape[1], _ptr(step.positions), B, n_chunks,
         cache.page_size, heads, kv_heads, head_dim, float(scale), int(window or 0), int(bool(write)), chunk,
-        cache.pages.shape[0], _status_ptr(dev), _stream()), "decode_attention_fused")
+        cache.pages.shape[0], _status_ptr(dev), int(q_map), _stream()), "decode_attention_fused")
     return out
 
 

@@ -44,8 +44,8 @@ Options that shape the scores or the values (they also take the one-product path
     d = o1 - lambda o2;   o = (1 - c) d / sqrt(mean(d^2) + eps) per head over Dv      (no weight), then Wo
 
 A page keeps a key head's two maps as one key of 2 D values, and a head's maps run as two query heads [q1 | 0] and [0 | q2]
-of the same key/value head: the zeros change no score, keys and values are cached and read once, and every attention
-kernel serves as it is.  One kernel combines the two outputs (`ops.attention_difference`).
+of the same key/value head (the kernels that read the projection's rows lay them out so: `q_map`): the zeros change no
+score, keys and values are cached and read once, and every attention kernel serves as it is.  One kernel combines the two outputs (`ops.attention_difference`).
 
 Reference: projections src/transformer/hybrid_attn.zig:285-354, per-head norm :371-382 (device
 :719,723), scale 1/sqrt(D) :571, causal mask :587, softmax :578-600, query head hq reads kv head
@@ -246,7 +246,6 @@ class Attention(Mixer):
         nm = self.names
         mats = [tensors[nm["q"]]]
         if self.differential is not None:
-            mats = [self._two_maps(tensors[nm["q"]])]
             vec = {k: tensors[nm[k]].double() for k in ("lq1", "lk1", "lq2", "lk2")}
             self.lam = float(torch.exp((vec["lq1"] * vec["lk1"]).sum()) - torch.exp((vec["lq2"] * vec["lk2"]).sum())) + self.differential
         if self.kv_proj:
@@ -269,14 +268,6 @@ class Attention(Mixer):
             self.w_o = torch.cat([w, w.new_zeros(self.hidden, self.heads, Dp - Dv)], dim=2).reshape(self.hidden, -1).contiguous()
         self.dtype = dtype
 
-    def _two_maps(self, q):
-        """The rows of a q projection [H, map 1 | map 2] as 2 H heads of 2 D rows: [map 1 | 0], [0 | map 2]."""
-        H, D = self.map_heads, self.map_dim
-        w = q.reshape(H, 2, D, self.hidden)
-        out = w.new_zeros((H, 2, 2, D, self.hidden))
-        out[:, 0, 0], out[:, 1, 1] = w[:, 0], w[:, 1]
-        return out.reshape(4 * H * D, self.hidden)
-
     def _output(self, o, ops):
         """From the heads' outputs [N, heads * cache_dim] through the output projection."""
         if self.differential is not None:
@@ -290,19 +281,21 @@ class Attention(Mixer):
         write = write_cache and self.kv_proj
         qkv = ops.linear(x, self.w_qkv)
         if self.value_norm or self.value_dim != self.head_dim:
-            qkv = ops.value_norm_pad(qkv, self.heads, self.kv_heads, self.head_dim, self.value_dim, self.eps, self.value_norm)
+            rows_heads = self.heads if self.differential is None else self.map_heads
+            qkv = ops.value_norm_pad(qkv, rows_heads, self.kv_heads, self.head_dim, self.value_dim, self.eps, self.value_norm)
         rot = self.position.rotary()
+        maps = {} if self.differential is None else {"q_map": self.map_dim}
         fused = getattr(ops, "fused_decode_attention_available", None)
         if (rot is not None and step.decode_only and self.kv_proj and fused is not None
                 and fused(qkv.dtype, self.heads, self.kv_heads, self.cache_dim)):
             # every row is one token: norm, rotation, page write, attention and the combination of
             # the key chunks run as one kernel
             o = ops.decode_attention_fused(qkv, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache,
-                                           self.heads, self.kv_heads, self.cache_dim, self.scale, self.window, write)
+                                           self.heads, self.kv_heads, self.cache_dim, self.scale, self.window, write, **maps)
             return self._output(o, ops)
         if rot is not None:
             q, _ = ops.qk_norm_rope(qkv, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache,
-                                    self.heads, self.kv_heads, self.cache_dim, self.kv_proj, write, False)
+                                    self.heads, self.kv_heads, self.cache_dim, self.kv_proj, write, False, **maps)
         else:
             q, k = ops.qk_norm_rope(qkv, self.q_norm, self.k_norm, self.norm_eps, 0, 1.0, step, cache,
                                     self.heads, self.kv_heads, self.cache_dim, self.kv_proj, False, self.kv_proj)
