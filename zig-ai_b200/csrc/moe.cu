@@ -26,12 +26,14 @@
 
 #define MOE_PLAIN_TN 64    // output columns of a block of the plain kernel
 #define MOE_PLAIN_TK 32    // k per stage of the plain kernel
-// Tiles of the tensor-core kernel by the tile height TM: output columns TN and warps of a block, k per stage, stages.  With few
-// rows a block mostly brings its weights in, one pass, so what it keeps in flight is what hides the way to memory.
-template <int TM> struct MoeTile {
-    static constexpr int TN = TM == 16 ? 32 : 64, WARPS = TM == 16 ? 2 : 4, TK = 64, ST = TK + 8, STAGES = TM == 16 ? 10 : 4;
+// The tensor-core kernel's block by the tile height TM and its output columns TN: warps, k per stage, stages.  With few rows a
+// block mostly brings its weights in, one pass, so what it keeps in flight is what hides the way to memory; narrow tiles
+// where wide ones would leave SMs without a block.  An output element is the same sum in the same order whatever TN is.
+template <int TM, int TN> struct MoeTile {
+    static constexpr int WARPS = TM == 16 ? TN / 16 : 4, TK = 64, ST = TK + 8, STAGES = TM == 16 ? (TN == 32 ? 10 : 6) : 4;
     static constexpr size_t BYTES = (size_t)STAGES * (TM + TN) * ST * 2;
 };
+#define MOE_WIDE_BLOCKS 296      // from this many blocks of 64 columns on, 64 columns a block
 
 // Eight neighbouring values as 32-bit numbers by 16-byte accesses (the caller has checked the alignment).
 __device__ __forceinline__ void moe_load8(float (&v)[8], const bf16* p) {
@@ -247,13 +249,13 @@ __device__ __forceinline__ int moe_weight_row(int r, int col_block, int n_out, i
     return f < n_out ? ((r >> 3) & 1) * n_out + f : -1;
 }
 
-template <int TM, typename TO>
-__global__ void __launch_bounds__(MoeTile<TM>::WARPS * 32) moe_gemm_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ xs,
+template <int TM, int TN, typename TO>
+__global__ void __launch_bounds__(MoeTile<TM, TN>::WARPS * 32) moe_gemm_mma_kernel(TO* __restrict__ out, const bf16* __restrict__ xs,
                                                            const bf16* __restrict__ w, const int* __restrict__ tile_expert,
                                                            int K, int n_out, int gated, const MoeAct act) {
-    constexpr int MOE_TN = MoeTile<TM>::TN, THREADS = MoeTile<TM>::WARPS * 32;
-    constexpr int WM = TM / 16, WN = MoeTile<TM>::WARPS / WM, NT = MOE_TN / 8 / WN;   // warps along rows and columns; 8-column tiles a warp
-    constexpr int MOE_TK = MoeTile<TM>::TK, MOE_ST = MoeTile<TM>::ST, MOE_STAGES = MoeTile<TM>::STAGES;
+    constexpr int MOE_TN = TN, THREADS = MoeTile<TM, TN>::WARPS * 32;
+    constexpr int WM = TM / 16, WN = MoeTile<TM, TN>::WARPS / WM, NT = MOE_TN / 8 / WN;   // warps along rows and columns; 8-column tiles a warp
+    constexpr int MOE_TK = MoeTile<TM, TN>::TK, MOE_ST = MoeTile<TM, TN>::ST, MOE_STAGES = MoeTile<TM, TN>::STAGES;
     extern __shared__ __align__(16) unsigned char moe_raw[];
     bf16 (*sa)[TM][MOE_ST] = reinterpret_cast<bf16 (*)[TM][MOE_ST]>(moe_raw);
     bf16 (*sb)[MOE_TN][MOE_ST] = reinterpret_cast<bf16 (*)[MOE_TN][MOE_ST]>(moe_raw + (size_t)MOE_STAGES * TM * MOE_ST * 2);
@@ -470,15 +472,15 @@ ZAI_API int zai_moe_gather(void* xs, int* dest, int* tile_expert, const void* x,
                                           max_tiles, scale_input));
 }
 
-template <int TM, typename TO>
+template <int TM, int TN, typename TO>
 static int moe_launch_mma(dim3 grid, TO* out, const bf16* xs, const bf16* w, const int* tile_expert, int K, int n_out, int gated,
                           const MoeAct& act, cudaStream_t stream) {
     static unsigned long long done = 0;
     if (zai_first_on_device(&done)) {
-        cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel<TM, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MoeTile<TM>::BYTES);
+        cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel<TM, TN, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MoeTile<TM, TN>::BYTES);
         if (e != cudaSuccess) return (int)e;
     }
-    return launch_pdl(moe_gemm_mma_kernel<TM, TO>, grid, dim3(MoeTile<TM>::WARPS * 32), MoeTile<TM>::BYTES, stream, out, xs, w, tile_expert, K, n_out, gated, act);
+    return launch_pdl(moe_gemm_mma_kernel<TM, TN, TO>, grid, dim3(MoeTile<TM, TN>::WARPS * 32), MoeTile<TM, TN>::BYTES, stream, out, xs, w, tile_expert, K, n_out, gated, act);
 }
 
 // out [max_tiles * TM, n_out] (32-bit if out_f32, else `dtype`) = xs [max_tiles * TM, K] . w[expert of the tile]^T;
@@ -492,13 +494,15 @@ ZAI_API int zai_moe_gemm(void* out, int out_f32, const void* xs, const void* w, 
     const int gated = kind == 1 || kind == 2;
     if (K < 1 || n_out < 1 || (TM != 16 && TM != 64)) return ZAI_BAD_SIZE;
     const bool mma = dtype == ZAI_BF16 && K % 8 == 0;
-    const int tn = mma ? (TM == 16 ? MoeTile<16>::TN : MoeTile<64>::TN) : MOE_PLAIN_TN, cols = gated ? tn / 2 : tn;
-    const dim3 grid(max_tiles, (n_out + cols - 1) / cols);
+    const auto blocks_of = [&](int tn) { const int cols = gated ? tn / 2 : tn; return (n_out + cols - 1) / cols; };
+    const bool wide = !mma || TM == 64 || (long long)max_tiles * blocks_of(64) >= MOE_WIDE_BLOCKS;
+    const dim3 grid(max_tiles, blocks_of(wide ? 64 : 32));
     if (grid.y > 65535) return ZAI_BAD_SIZE;
     if (mma) {
-#define MOE_GO(TMV, TOV) return moe_launch_mma<TMV, TOV>(grid, (TOV*)out, (const bf16*)xs, (const bf16*)w, tile_expert, K, n_out, gated, act, stream)
-        if (TM == 16) { if (out_f32) MOE_GO(16, float); else MOE_GO(16, bf16); }
-        if (out_f32) MOE_GO(64, float); else MOE_GO(64, bf16);
+#define MOE_GO(TMV, TNV, TOV) return moe_launch_mma<TMV, TNV, TOV>(grid, (TOV*)out, (const bf16*)xs, (const bf16*)w, tile_expert, K, n_out, gated, act, stream)
+        if (TM == 64) { if (out_f32) MOE_GO(64, 64, float); else MOE_GO(64, 64, bf16); }
+        if (wide) { if (out_f32) MOE_GO(16, 64, float); else MOE_GO(16, 64, bf16); }
+        if (out_f32) MOE_GO(16, 32, float); else MOE_GO(16, 32, bf16);
 #undef MOE_GO
     }
     if (TM != 16) return ZAI_BAD_SIZE;                   // the plain kernel's tiles are 16 rows high
