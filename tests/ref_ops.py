@@ -81,6 +81,21 @@ def add_rmsnorm(h, delta, w, eps, out_dtype, delta_gamma=None, delta_eps=0.0):
     return (h * torch.rsqrt(ms + eps) * _f(w)).to(out_dtype)
 
 
+def add_rmsnorm_pair(h, delta, w_a, w_b, eps, out_dtype, delta_gamma=None, delta_eps=0.0):
+    a = add_rmsnorm(h, delta, w_a, eps, out_dtype, delta_gamma, delta_eps)
+    return a, add_rmsnorm(h, None, w_b, eps, out_dtype)
+
+
+def linear_add(x, w, addend):
+    return _f(x) @ _f(w).T + addend
+
+
+def linear_side(x, w, table, ids, at):
+    """gelu_tanh(x . w^T) times columns at .. of the rows' entries in a table by token id."""
+    rows = _f(table[_checked(ids.long(), table.shape[0], 2)][:, at:at + w.shape[0]])
+    return (activation(_f(linear(x, w)), "gelu_tanh") * rows).to(x.dtype)
+
+
 def linear(x, w, out_dtype=None, bias=None):
     out_dtype = out_dtype or x.dtype
     if bias is not None:
@@ -246,9 +261,11 @@ def paged_attention(q, step, cache, heads, kv_heads, head_dim, scale, window=Non
     return out
 
 
-def add_cast(h, delta, out_dtype, delta_gamma=None, delta_eps=0.0):
+def add_cast(h, delta, out_dtype, delta_gamma=None, delta_eps=0.0, delta2=None):
     if delta is not None:
         h += _f(delta) if delta_gamma is None else _normed(delta, delta_gamma, delta_eps)
+    if delta2 is not None:
+        h += _f(delta2)
     return h.to(out_dtype) if out_dtype != h.dtype else h.clone()
 
 
@@ -528,9 +545,12 @@ def qkv_prepare(y, q_w, k_w, eps, scope, table, rot, step, cache, heads, kv_head
     return pad(q, Dp).to(y.dtype).reshape(N, H * Dp)
 
 
-def sigmoid_gate(o, gate, heads, head_dim, per_head):
-    """o [N, heads * head_dim] times sigmoid(gate): gate [N, heads] (one number per head) or [N, heads * head_dim]."""
+def sigmoid_gate(o, gate, heads, head_dim, per_head, row_dim=None):
+    """o [N, heads * head_dim] times sigmoid(gate): gate [N, heads] (one number per head) or [N, heads * head_dim].  `row_dim`:
+    the heads lie that far apart in o's rows."""
     N = o.shape[0]
+    if row_dim is not None:
+        o = o.reshape(N, heads, row_dim)[:, :, :head_dim].reshape(N, heads * head_dim)
     g = torch.sigmoid(_f(gate))
     if per_head:
         return (_f(o).reshape(N, heads, head_dim) * g[:, :, None]).reshape(N, heads * head_dim).to(o.dtype)
@@ -608,24 +628,38 @@ def rmsnorm_rows(x, w, eps):
 
 
 def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on="input", score="sigmoid", act="silu", limit=0.0,
-                   alpha=1.702, router_bias=None, unit=None, unit_gated=False):
+                   alpha=1.702, router_bias=None, unit=None, unit_gated=False, correction=None, groups=None, identities=0,
+                   weight_scale=1.0, onto=None):
     """Every row to the `top` experts with the largest sigmoid(x . w_router^T); the scores weigh the experts' inputs
-    or outputs; w_gate_up [E, 2F, W] (gate rows, then up rows; [E, F, W] for "relu2"), w_down [E, W, F]."""
+    or outputs; w_gate_up [E, 2F, W] (gate rows, then up rows; [E, F, W] for "relu2"), w_down [E, W, F].  `correction`, `groups`
+    (count, keep) change the choice alone; the last `identities` outputs of the router give the row itself."""
     N, W = x.shape
     E, F = w_gate_up.shape[0], w_gate_up.shape[1] // (1 if act == "relu2" else 2)
+    A = E + int(identities)
     z = _f(x) @ _f(w_router).t()
-    gate = torch.sigmoid(z[:, E:]) if unit_gated else None
-    z = z[:, :E] if router_bias is None else z[:, :E] + router_bias
+    gate = torch.sigmoid(z[:, A:]) if unit_gated else None
+    z = z[:, :A] if router_bias is None else z[:, :A] + router_bias
     s = torch.softmax(z, dim=-1) if score == "softmax" else z if score == "chosen" else torch.sigmoid(z)
-    val, idx = torch.topk(s, int(top), dim=-1)
+    choice = s if correction is None else s + correction
+    if groups is not None:
+        best = choice.reshape(N, groups[0], -1).max(dim=-1).values
+        order = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, :groups[1]]
+        kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, order, True).repeat_interleave(A // groups[0], dim=1)
+        choice = choice.masked_fill(~kept, float("-inf"))
+    _, idx = torch.topk(choice, int(top), dim=-1)
+    val = torch.gather(s, 1, idx)
     if score == "chosen":
         val = torch.softmax(val, dim=-1)
     if renorm:
         val = val / (val.sum(-1, keepdim=True) + 1e-20)
+    val = val * weight_scale
     out = torch.zeros((N, W), dtype=torch.float32, device=x.device)
     for n in range(N):
         for k in range(int(top)):
             e, w = int(idx[n, k]), val[n, k]
+            if e >= E:
+                out[n] += w * _f(x[n])
+                continue
             xin = (_f(x[n]) * w).to(x.dtype) if weight_on == "input" else x[n]
             gu = _f(xin) @ _f(w_gate_up[e]).t()
             if act == "relu2":
@@ -639,6 +673,10 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
             out[n] += y if weight_on == "input" else y * w
     if unit is not None:
         out += _f(unit) if gate is None else gate * _f(unit)
+    if onto is not None:
+        h, other, cast = onto
+        h += out if other is None else out + _f(other)
+        return h.to(x.dtype).clone() if cast else None
     return out.to(x.dtype)
 
 

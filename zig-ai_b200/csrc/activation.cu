@@ -80,6 +80,35 @@ ZAI_API int zai_act_mul(void* out, const void* gu, int dtype, int N, int F, int 
     ZAI_DISPATCH(dtype, return launch_pdl(act_mul_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)out, (const T*)gu, F, total, kind));
 }
 
+// act(x) times the row's entries of a table, looked up by token id: out[t, d] = act(x[t, d]) * table[ids[t], at + d]
+template <typename T>
+__global__ void act_mul_rows_kernel(T* __restrict__ out, const T* __restrict__ x, const T* __restrict__ table, const int* __restrict__ ids,
+                                    int rows, int ld, int at, int D, size_t total, int kind, int* __restrict__ status) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const size_t t = i / D;
+    const int d = (int)(i - t * D);
+    int id = ids[t];
+    if ((unsigned)id >= (unsigned)rows) {
+        zai_raise(status, ZAI_ST_TOKEN);
+        id = 0;
+    }
+    out[i] = from_float<T>(zai_activate(to_float(x[i]), kind) * to_float(table[(size_t)id * ld + at + d]));
+}
+
+// x [N, D], table [rows, ld]; an id outside the table counts as 0 and raises the status word
+ZAI_API int zai_act_mul_rows(void* out, const void* x, const void* table, const int* ids, int rows, int ld, int at, int dtype, int N, int D,
+                             int kind, int* status, cudaStream_t stream) {
+    const size_t total = (size_t)N * D;
+    if (N <= 0 || total == 0) return ZAI_OK;
+    if (kind < 0 || kind > 4 || rows < 1 || at < 0 || at + D > ld) return ZAI_BAD_SIZE;
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    ZAI_DISPATCH(dtype, return launch_pdl(act_mul_rows_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)out, (const T*)x, (const T*)table,
+                                          ids, rows, ld, at, D, total, kind, status));
+}
+
 template <typename T>
 __global__ void activation_kernel(T* __restrict__ out, const T* __restrict__ in, int kind, size_t total) {
     pdl_trigger();

@@ -86,7 +86,13 @@ struct SkinnyArgs {
     // the scaled sums
     int center;
     const float* beta_dot;
-    int plain_act;        // bfloat16 epilogue: 1: y = relu(.)^2, 0: as it is
+    int plain_act;        // bfloat16 epilogue: 1: y = relu(.)^2, 2: y = gelu_tanh(.) * side row, 0: as it is
+    const bf16* bias;     // [O] added to the sums, or null (bfloat16 and 32-bit epilogues)
+    const float* addend;  // 32-bit epilogue: [M, O] added to the sums, or null
+    // plain_act 2: token m's row of a table [side_rows, side_ld], columns side_at .. side_at + O - 1 (an id outside: row 0, status)
+    const bf16* side;
+    const int* side_ids;
+    int side_rows, side_ld, side_at;
 };
 
 __device__ __forceinline__ void cp_async16_zfill(void* smem, const void* gmem, bool valid) {
@@ -114,6 +120,8 @@ __device__ __forceinline__ void mma16816(float (&d)[4], uint32_t a0, uint32_t a1
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
+
+__device__ __forceinline__ float sg_gelu_tanh(float z) { return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z))); }
 
 // Blocks are persistent: block b takes the work units b, b + gridDim.x, ...; a unit is `tpc` tiles of
 // 16 weight rows, each tile's K cut into `sk` slices, one slice per warp (8 warps).  A block uses
@@ -508,6 +516,10 @@ __global__ void __launch_bounds__(SG_WARPS * 32, 2) skinny_gemm_kernel(const Ski
                     if (row_lo >= 0) lo += a.beta_dot[row_lo];
                     if (row_hi >= 0) hi += a.beta_dot[row_hi];
                 }
+                if (EPI != EPI_SWIGLU && a.bias) {
+                    if (row_lo >= 0) lo += __bfloat162float(a.bias[row_lo]);
+                    if (row_hi >= 0) hi += __bfloat162float(a.bias[row_hi]);
+                }
                 if (EPI == EPI_SWIGLU) {
                     if (row_lo >= 0) {
                         float gt = lo, up = hi, slope = 1.f;
@@ -517,15 +529,28 @@ __global__ void __launch_bounds__(SG_WARPS * 32, 2) skinny_gemm_kernel(const Ski
                             slope = a.glu_slope;
                         }
                         const float act = a.glu_limit < 0.f          // (a negative limit: the gate passes the tanh form of GELU)
-                            ? 0.5f * lo * (1.f + tanhf(0.79788456080286536f * (lo + 0.044715f * lo * lo * lo)))
+                            ? sg_gelu_tanh(lo)
                             : gt / (1.f + expf(-slope * gt));
                         reinterpret_cast<bf16*>(a.y)[(size_t)tok * a.ldy + row_lo] = __float2bfloat16_rn(act * up);
                     }
                 } else if (EPI == EPI_F32) {
+                    if (a.addend) {
+                        if (row_lo >= 0) lo += a.addend[(size_t)tok * a.O + row_lo];
+                        if (row_hi >= 0) hi += a.addend[(size_t)tok * a.O + row_hi];
+                    }
                     if (row_lo >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.ldy + row_lo] = lo;
                     if (row_hi >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.ldy + row_hi] = hi;
                 } else {
-                    if (EPI == EPI_BF16 && a.plain_act) {
+                    if (EPI == EPI_BF16 && a.plain_act == 2) {
+                        int id = a.side_ids[tok];
+                        if ((unsigned)id >= (unsigned)a.side_rows) {
+                            zai_raise(a.status, ZAI_ST_TOKEN);
+                            id = 0;
+                        }
+                        const bf16* s = a.side + (size_t)id * a.side_ld + a.side_at;
+                        if (row_lo >= 0) lo = sg_gelu_tanh(lo) * __bfloat162float(s[row_lo]);
+                        if (row_hi >= 0) hi = sg_gelu_tanh(hi) * __bfloat162float(s[row_hi]);
+                    } else if (EPI == EPI_BF16 && a.plain_act) {
                         lo = fmaxf(lo, 0.f) * fmaxf(lo, 0.f);
                         hi = fmaxf(hi, 0.f) * fmaxf(hi, 0.f);
                     }
@@ -556,6 +581,8 @@ struct SplitKArgs {
     int M, O, K, n_tiles;
     int per;              // 32-k blocks per warp
     int f32_out;
+    const bf16* bias;     // [O] added to the sums, or null
+    const float* addend;  // [M, O] added to the sums, or null (32-bit results)
     NextWeights next;
 };
 
@@ -670,7 +697,15 @@ __global__ void __launch_bounds__(SG_WARPS * 32) skinny_splitk_kernel(const Spli
         for (int e = 0; e < 2; ++e) {
             const int tok = nt * 8 + 2 * t + e;
             if (tok >= a.M) continue;
-            const float lo = c[nt][e], hi = c[nt][2 + e];
+            float lo = c[nt][e], hi = c[nt][2 + e];
+            if (a.bias) {
+                if (row_lo >= 0) lo += __bfloat162float(a.bias[row_lo]);
+                if (row_hi >= 0) hi += __bfloat162float(a.bias[row_hi]);
+            }
+            if (a.addend) {
+                if (row_lo >= 0) lo += a.addend[(size_t)tok * a.O + row_lo];
+                if (row_hi >= 0) hi += a.addend[(size_t)tok * a.O + row_hi];
+            }
             if (a.f32_out) {
                 if (row_lo >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.O + row_lo] = lo;
                 if (row_hi >= 0) reinterpret_cast<float*>(a.y)[(size_t)tok * a.O + row_hi] = hi;
@@ -891,7 +926,9 @@ static int skinny_run(SkinnyArgs& a, int epilogue, cudaStream_t stream) {
 static int skinny_gemm_run(void* y, const void* W, const void* x, const float* h, const void* delta,
                            const float* gamma, const int* row_idx, float* h_out, float eps, int M, int O, int K,
                            int epilogue, float glu_limit, float glu_slope, cudaStream_t stream, int center = 0,
-                           const float* beta_dot = nullptr, int plain_act = 0) {
+                           const float* beta_dot = nullptr, int plain_act = 0, const void* bias = nullptr,
+                           const float* addend = nullptr, const SkinnyArgs* side = nullptr) {
+    if ((addend && epilogue != EPI_F32) || (bias && epilogue == EPI_SWIGLU) || (plain_act == 2 && !side)) return ZAI_BAD_SIZE;
     if (epilogue == EPI_CONV || !zai_skinny_gemm_supports(M, O, K, epilogue, h != nullptr)) return ZAI_BAD_SIZE;
     const int cs = (!h && !plain_act && (epilogue == EPI_BF16 || epilogue == EPI_F32)) ? splitk_cluster(K) : 0;
     if (cs) {
@@ -900,11 +937,14 @@ static int skinny_gemm_run(void* y, const void* W, const void* x, const float* h
         b.n_tiles = (O + 15) / 16;
         b.per = ((K + 31) / 32 + SG_WARPS * cs - 1) / (SG_WARPS * cs);
         b.f32_out = epilogue == EPI_F32;
+        b.bias = (const bf16*)bias; b.addend = addend;
         if (cs == 8) return M <= 8 ? splitk_launch<1, 8>(b, stream) : splitk_launch<2, 8>(b, stream);
         if (cs == 4) return M <= 8 ? splitk_launch<1, 4>(b, stream) : splitk_launch<2, 4>(b, stream);
         return M <= 8 ? splitk_launch<1, 2>(b, stream) : splitk_launch<2, 2>(b, stream);
     }
     SkinnyArgs a = {};
+    if (side) { a.side = side->side; a.side_ids = side->side_ids; a.side_rows = side->side_rows; a.side_ld = side->side_ld; a.side_at = side->side_at; a.status = side->status; }
+    a.bias = (const bf16*)bias; a.addend = addend;
     a.W = (const bf16*)W; a.x = (const bf16*)x; a.h = h; a.delta = (const bf16*)delta; a.gamma = gamma;
     a.row_idx = row_idx; a.h_out = h_out; a.y = y; a.eps = eps; a.M = M; a.O = O; a.K = K;
     a.F = O / 2;
@@ -951,6 +991,26 @@ ZAI_API int zai_skinny_gemm_clamped_glu(void* y, const void* W, const void* x, c
 ZAI_API int zai_skinny_gemm_relu2(void* y, const void* W, const void* x, const float* h, const void* delta, const float* gamma,
                                   const int* row_idx, float* h_out, float eps, int M, int O, int K, cudaStream_t stream) {
     return skinny_gemm_run(y, W, x, h, delta, gamma, row_idx, h_out, eps, M, O, K, EPI_BF16, 0.f, 1.f, stream, 0, nullptr, 1);
+}
+
+// y = x . W^T + bias (bfloat16 [O]; epilogue 0 or 1), or, in 32-bit (epilogue 1), + addend [M, O]; x or a norm of h as above
+// (`beta_dot`: a layer norm's, else an RMS norm's).
+ZAI_API int zai_skinny_gemm_added(void* y, const void* W, const void* x, const float* h, const void* delta, const float* gamma,
+                                  const float* beta_dot, const int* row_idx, float* h_out, float eps, int M, int O, int K, int epilogue,
+                                  const void* bias, const float* addend, cudaStream_t stream) {
+    if (epilogue != EPI_BF16 && epilogue != EPI_F32) return ZAI_BAD_SIZE;
+    return skinny_gemm_run(y, W, x, h, delta, gamma, row_idx, h_out, eps, M, O, K, epilogue, 0.f, 1.f, stream, beta_dot != nullptr, beta_dot,
+                           0, bias, addend);
+}
+
+// y = gelu_tanh(x . W^T) * table[ids[m], at .. at + O - 1], bfloat16 [M, O]; table [rows, ld] bfloat16.
+ZAI_API int zai_skinny_gemm_side(void* y, const void* W, const void* x, int M, int O, int K, const void* table, const int* ids, int rows,
+                                 int ld, int at, int* status, cudaStream_t stream) {
+    if (rows < 1 || at < 0 || at + O > ld) return ZAI_BAD_SIZE;
+    SkinnyArgs side = {};
+    side.side = (const bf16*)table; side.side_ids = ids; side.side_rows = rows; side.side_ld = ld; side.side_at = at; side.status = status;
+    return skinny_gemm_run(y, W, x, nullptr, nullptr, nullptr, nullptr, nullptr, 0.f, M, O, K, EPI_BF16, 0.f, 1.f, stream, 0, nullptr, 2,
+                           nullptr, nullptr, &side);
 }
 
 // The short convolution's input projection with the convolution as its epilogue, for steps in which

@@ -6,6 +6,11 @@
 //   y = sum over the chosen e of  down_e( silu(gate_e(x_e)) * up_e(x_e) ),   x_e = w_e x   (`weight_on` input)
 //                                or of  w_e down_e( silu(gate_e(x)) * up_e(x) )             (`weight_on` output)
 //
+// The choice may differ from the scores: choice = s + a correction per expert, the experts may form groups of neighbours of
+// which only the best few (by their largest choice value) are chosen from, and the weights may be multiplied by a factor.  The
+// last experts of the router may be identities: they have no matrices and give the row itself, so their rows never enter the
+// sorted layout and join in the combine.
+//
 // The experts may also be units without a gate, down_e( act(up_e(x)) ), act the square of relu; and a unit that every row
 // passes beside its experts joins in the combine, weighed by the sigmoid of one more 32-bit product of the row.
 //
@@ -19,7 +24,8 @@
 //     tile of TM rows x 32 or 64 output columns of one expert; bfloat16 on the tensor cores (mma.sync m16n8k16, cp.async
 //     ring), any other case by 32-bit multiply-adds.  Steps with many rows an expert gather with a
 //     tile height of 128 and run both products in the grouped mode of the tcgen05 kernel (gemm_tc.cu) instead;
-//   * combine: a row's `top` results summed in 32-bit in the order of the choice and rounded once.
+//   * combine: a row's `top` results summed in 32-bit in the order of the choice and rounded once; or the sum, unrounded, and
+//     the rows of a mixer beside the experts are added to the 32-bit residual stream, which is then rounded for its next reader.
 // A row's result depends on the row alone: on which tile it lands, what else the tile holds and in which order the
 // counter was taken changes nothing, since every output element is a sum over k in a fixed order.
 #include "mma_helpers.cuh"
@@ -67,14 +73,23 @@ __device__ __forceinline__ bool moe_rows_aligned(const T* p, size_t stride, int 
 
 // ------------------------------------------------------------------------------------------------ route
 enum { MOE_SIGMOID = 0, MOE_SOFTMAX = 1, MOE_LOGITS = 2 };          // what the scores are
+// How the choice differs from the scores (all zero: it does not).  `real`: the experts that have matrices; those behind them
+// are identities.
+struct MoeChoice {
+    const float* correction;       // [E] or null
+    int groups, keep, real;        // groups 0: none
+    float scale;                   // on the weights
+    __host__ __device__ bool own() const { return correction != nullptr || groups > 0; }      // a choice value beside the score
+};
 // ROWS rows a block (their values are read once per expert row of the router for all of them); a row's sums have the same order
 // whatever ROWS and the number of warps are.
 template <typename T, int ROWS>
 __global__ void __launch_bounds__(512) moe_route_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ rank,
                                                         int* __restrict__ counts, const T* __restrict__ x, int x_stride,
                                                         const float* __restrict__ wr, int N, int W, int E, int top, int renorm,
-                                                        int score, const float* __restrict__ bias, float* __restrict__ unit_gate) {
-    extern __shared__ float sc_all[];                    // [ROWS][E] scores
+                                                        int score, const float* __restrict__ bias, float* __restrict__ unit_gate,
+                                                        const MoeChoice choice) {
+    extern __shared__ float sc_all[];                    // [ROWS][E] scores, then (a choice of its own) [ROWS][E + groups]
     const int tr = blockIdx.x * ROWS, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     pdl_trigger();
     pdl_wait();
@@ -126,12 +141,35 @@ __global__ void __launch_bounds__(512) moe_route_kernel(int* __restrict__ ids, f
         for (int e = lane; e < E; e += 32) sc[e] = expf(sc[e] - top_z) / total;
         __syncwarp();
     }
+    float* ch = sc;                                      // what the choice goes by
+    if (choice.own()) {
+        ch = sc_all + ROWS * E + warp * (E + choice.groups);
+        for (int e = lane; e < E; e += 32) ch[e] = choice.correction ? sc[e] + choice.correction[e] : sc[e];
+        __syncwarp();
+        if (choice.groups > 0) {                         // a group's value is its largest; the `keep` best groups stay (ties: the lower)
+            float* gv = ch + E;
+            const int size = E / choice.groups;
+            for (int q = lane; q < choice.groups; q += 32) {
+                float v = ch[q * size];
+                for (int i = 1; i < size; ++i) v = fmaxf(v, ch[q * size + i]);
+                gv[q] = v;
+            }
+            __syncwarp();
+            for (int q = lane; q < choice.groups; q += 32) {
+                int above = 0;
+                for (int o = 0; o < choice.groups; ++o) above += gv[o] > gv[q] || (gv[o] == gv[q] && o < q);
+                if (above >= choice.keep)
+                    for (int i = 0; i < size; ++i) ch[q * size + i] = -INFINITY;
+            }
+            __syncwarp();
+        }
+    }
     float sum = 0.f, mine = -INFINITY, first = 0.f;      // (`mine`: lane k keeps the k-th choice's score)
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = sc[e];
+            const float v = ch[e];
             if (v > best) { best = v; at = e; }          // (ascending e: the first of equals stays)
         }
 #pragma unroll
@@ -141,11 +179,13 @@ __global__ void __launch_bounds__(512) moe_route_kernel(int* __restrict__ ids, f
             if (ov > best || (ov == best && oa < at)) { best = ov; at = oa; }
         }
         if (at >= E) at = 0;                             // (scores that are no numbers: any expert, never an index outside)
+        if (choice.own()) best = sc[at];                 // the weight is the score, whatever the choice went by
+        __syncwarp();
         if (lane == 0) {
             ids[(size_t)t * top + k] = at;
             wts[(size_t)t * top + k] = best;
-            rank[(size_t)t * top + k] = atomicAdd(&counts[at], 1);
-            sc[at] = -INFINITY;
+            rank[(size_t)t * top + k] = at < choice.real ? atomicAdd(&counts[at], 1) : -1;
+            ch[at] = -INFINITY;
         }
         if (lane == k) mine = best;
         if (k == 0) first = best;
@@ -159,7 +199,9 @@ __global__ void __launch_bounds__(512) moe_route_kernel(int* __restrict__ ids, f
         if (lane < top) wts[(size_t)t * top + lane] = w / total;
         return;
     }
-    if (renorm && lane < top) wts[(size_t)t * top + lane] /= sum + 1e-20f;
+    if (lane >= top) return;
+    if (renorm) wts[(size_t)t * top + lane] = wts[(size_t)t * top + lane] / (sum + 1e-20f) * choice.scale;
+    else if (choice.scale != 1.f) wts[(size_t)t * top + lane] *= choice.scale;
 }
 
 // ------------------------------------------------------------------------------------------------ gather
@@ -190,6 +232,10 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(T* __restrict__ xs, int
         return;
     }
     const int item = blockIdx.x, t = item / top, e = ids[item];
+    if (e >= E) {                                        // an identity: nothing to sort
+        if (threadIdx.x == 0) dest[item] = -1;
+        return;
+    }
     float before = 0.f;                                  // (whole numbers below 2^24: exact in 32-bit floats)
     for (int o = threadIdx.x; o < e; o += blockDim.x) before += (float)(((counts[o] + TM - 1) / TM) * TM);
     const int first = (int)block_sum(before, red);
@@ -393,42 +439,76 @@ __global__ void __launch_bounds__(128) moe_gemm_plain_kernel(TO* __restrict__ ou
 }
 
 // ------------------------------------------------------------------------------------------------ combine
+// What the combine adds beside the experts' results.  `h`: the residual stream [N, W]; the row's sum and `other` (the rows of
+// a mixer that read the same stream, or null) are added to it and `out` (which may then be null) gets the stream rounded.
+template <typename T>
+struct MoeBeside {
+    const T* unit;                 // [N, W] rows of the unit beside the experts, or null
+    const float* unit_gate;        // [N] its weights, or null
+    const T* x;                    // the rows that identities give (dest < 0), row stride x_stride
+    int x_stride;
+    float* h;
+    const T* other;
+};
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ y, const int* __restrict__ dest,
-                                   const float* __restrict__ wts, int W, int top, int scale_output, const T* __restrict__ unit,
-                                   const float* __restrict__ unit_gate) {
+                                   const float* __restrict__ wts, int W, int top, int scale_output, const MoeBeside<T> a) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
-    const float ug = unit_gate ? unit_gate[t] : 1.f;     // (`unit`: the rows of the unit beside the experts)
-    if ((W & 7) == 0 && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(unit)) & 15) == 0) {
+    const float ug = a.unit_gate ? a.unit_gate[t] : 1.f;
+    const T* xrow = a.x ? a.x + (size_t)t * a.x_stride : nullptr;
+    const uintptr_t addresses = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(a.unit) |
+                                reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.h) | reinterpret_cast<uintptr_t>(a.other);
+    if ((W & 7) == 0 && (addresses & 15) == 0 && (a.x_stride & 7) == 0) {
         for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {      // the same sums in the same order, eight columns at a time
             float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             for (int k = 0; k < top; ++k) {
                 float v[8];
-                moe_load8(v, y + (size_t)dest[(size_t)t * top + k] * W + c);
-                const float wk = scale_output ? wts[(size_t)t * top + k] : 1.f;
+                const int d = dest[(size_t)t * top + k];
+                if (d >= 0) moe_load8(v, y + (size_t)d * W + c);
+                else moe_load8(v, xrow + c);
+                const bool scaled = scale_output || d < 0;
+                const float wk = scaled ? wts[(size_t)t * top + k] : 1.f;
 #pragma unroll
-                for (int i = 0; i < 8; ++i) acc[i] += scale_output ? v[i] * wk : v[i];
+                for (int i = 0; i < 8; ++i) acc[i] += scaled ? v[i] * wk : v[i];
             }
-            if (unit) {
+            if (a.unit) {
                 float v[8];
-                moe_load8(v, unit + (size_t)t * W + c);
+                moe_load8(v, a.unit + (size_t)t * W + c);
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[i] += ug * v[i];
             }
-            moe_store8(out + (size_t)t * W + c, acc);
+            if (a.h) {
+                float v[8];
+                if (a.other) {
+                    moe_load8(v, a.other + (size_t)t * W + c);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) acc[i] += v[i];
+                }
+                moe_load8(v, a.h + (size_t)t * W + c);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[i] += v[i];
+                moe_store8(a.h + (size_t)t * W + c, acc);
+            }
+            if (out) moe_store8(out + (size_t)t * W + c, acc);
         }
         return;
     }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
-            const float v = y[(size_t)dest[(size_t)t * top + k] * W + c];
-            acc += scale_output ? v * wts[(size_t)t * top + k] : v;
+            const int d = dest[(size_t)t * top + k];
+            const float v = d >= 0 ? y[(size_t)d * W + c] : to_float(xrow[c]);
+            acc += scale_output || d < 0 ? v * wts[(size_t)t * top + k] : v;
         }
-        if (unit) acc += ug * to_float(unit[(size_t)t * W + c]);
-        out[(size_t)t * W + c] = from_float<T>(acc);
+        if (a.unit) acc += ug * to_float(a.unit[(size_t)t * W + c]);
+        if (a.h) {
+            if (a.other) acc += to_float(a.other[(size_t)t * W + c]);
+            acc += a.h[(size_t)t * W + c];
+            a.h[(size_t)t * W + c] = acc;
+        }
+        if (out) out[(size_t)t * W + c] = from_float<T>(acc);
     }
 }
 
@@ -436,21 +516,28 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
 // ids, rank [N, top] int; wts [N, top] 32-bit; counts [E] int, zeroed here; x [N, x_stride] in `dtype`; wr [E, W] 32-bit.
 // score: 0 sigmoid, 1 softmax over all experts, 2 the logits with softmax over the chosen (`bias` [E] 32-bit or null is added to
 // the logits; modes 1 and 2).  With `unit_gate` [N] wr has one row more, whose product's sigmoid goes there.
+// E counts identities too; `real` of them have matrices (and counts).  `correction` [E] or null, `groups` (0: none) of which `keep`
+// are chosen from, `scale` on the weights: see MoeChoice.
 ZAI_API int zai_moe_route(int* ids, float* wts, int* rank, int* counts, const void* x, int x_stride, int dtype, const float* wr,
                           int N, int W, int E, int top, int renorm, int score, const float* bias, float* unit_gate,
-                          cudaStream_t stream) {
+                          const float* correction, int groups, int keep, int real, float scale, cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
+    const MoeChoice choice = {correction, groups, keep, real, scale};
+    if (real < 1 || real > E || groups < 0 || (groups && (E % groups || keep < 1 || keep > groups || (long long)keep * (E / groups) < top))
+        || (score == MOE_LOGITS && (choice.own() || scale != 1.f)) || (choice.own() && E > 4096)) return ZAI_BAD_SIZE;
     if (E < 1 || top < 1 || top > E || top > 32 || E > 8192 || W < 1 || score < MOE_SIGMOID || score > MOE_LOGITS || (bias && score == MOE_SIGMOID)) return ZAI_BAD_SIZE;
-    cudaError_t rc = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int), stream);
+    cudaError_t rc = cudaMemsetAsync(counts, 0, (size_t)real * sizeof(int), stream);
     if (rc != cudaSuccess) return (int)rc;
     const int rows = E + (unit_gate ? 1 : 0);
-    if (N >= 512 && E <= 2048) {
-        ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 4>, dim3((N + 3) / 4), dim3(rows <= 4 ? 128 : 256), (size_t)4 * E * sizeof(float),
-                                              stream, ids, wts, rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate));
+    const size_t smem = (size_t)(E + (choice.own() ? E + groups : 0)) * sizeof(float);      // a row's scores and choice values
+    if (N >= 512 && 4 * smem <= 32 * 1024) {
+        ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 4>, dim3((N + 3) / 4), dim3(rows <= 4 ? 128 : 256), 4 * smem,
+                                              stream, ids, wts, rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate,
+                                              choice));
     }
     const int warps = rows < 4 ? 4 : rows > 16 ? 16 : rows;
-    ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 1>, dim3(N), dim3(warps * 32), (size_t)E * sizeof(float), stream, ids, wts,
-                                          rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate));
+    ZAI_DISPATCH(dtype, return launch_pdl(moe_route_kernel<T, 1>, dim3(N), dim3(warps * 32), smem, stream, ids, wts,
+                                          rank, counts, (const T*)x, x_stride, wr, N, W, E, top, renorm, score, bias, unit_gate, choice));
 }
 
 // The most tiles of TM rows that N x top choices over E experts can take.
@@ -518,10 +605,14 @@ ZAI_API int zai_moe_gemm(void* out, int out_f32, const void* xs, const void* w, 
 }
 
 // out [N, W] in `dtype` = sum over a row's choices of y[dest], times the choice's weight with `scale_output`; plus, with `unit`
-// [N, W] in `dtype`, that row times unit_gate[row] (32-bit; null: times 1)
+// [N, W] in `dtype`, that row times unit_gate[row] (32-bit; null: times 1).  A choice with dest < 0 gives its weight times the
+// row of x (may be null where there is none).  With `h` [N, W] 32-bit: h += that sum + other (or null), out (or null) = h rounded.
 ZAI_API int zai_moe_combine(void* out, int dtype, const float* y, const int* dest, const float* wts, int N, int W, int top,
-                            int scale_output, const void* unit, const float* unit_gate, cudaStream_t stream) {
+                            int scale_output, const void* unit, const float* unit_gate, const void* x, int x_stride, float* h,
+                            const void* other, cudaStream_t stream) {
     if (N <= 0) return ZAI_OK;
-    ZAI_DISPATCH(dtype, return launch_pdl(moe_combine_kernel<T>, dim3(N), dim3(W >= 1024 ? 256 : 128), 0, stream, (T*)out, y, dest,
-                                          wts, W, top, scale_output, (const T*)unit, unit_gate));
+    if (!out && !h) return ZAI_BAD_SIZE;
+    ZAI_DISPATCH(dtype, const MoeBeside<T> a = {(const T*)unit, unit_gate, (const T*)x, x_stride, h, (const T*)other};
+                 return launch_pdl(moe_combine_kernel<T>, dim3(N), dim3(W >= 1024 ? 256 : 128), 0, stream, (T*)out, y, dest, wts, W, top,
+                                   scale_output, a));
 }

@@ -34,13 +34,14 @@ _SIGNATURES = {
     },
     "norm": {"zai_add_rmsnorm": [_P, _P, _P, _P, _I, _F, _I, _I, _P],
              "zai_add_normed_rmsnorm": [_P, _P, _P, _F, _P, _P, _I, _F, _I, _I, _P],
-             "zai_add_normed_cast": [_P, _P, _P, _F, _P, _I, _I, _I, _P],
+             "zai_add_rmsnorm_pair": [_P, _P, _P, _F, _P, _P, _P, _P, _I, _F, _I, _I, _P],
+             "zai_add_normed_cast": [_P, _P, _P, _F, _P, _I, _I, _I, _P, _P],
              "zai_rmsnorm_rows": [_P, _P, _I, _I, _P, _F, _I, _I, _P]},
-    "moe": {"zai_moe_route": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P],
+    "moe": {"zai_moe_route": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _F, _P],
             "zai_moe_max_tiles": [_I, _I, _I, _I],
             "zai_moe_gather": [_P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
             "zai_moe_gemm": [_P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _P],
-            "zai_moe_combine": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P]},
+            "zai_moe_combine": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P]},
     "attention_difference": {"zai_attention_difference": [_P, _P, _I, _F, _F, _F, _I, _I, _I, _I, _P]},
     "mamba2": {
         "zai_mamba2_chunked_supports": [_I, _I],
@@ -65,6 +66,7 @@ _SIGNATURES = {
     "activation": {"zai_silu_mul": [_P, _P, _I, _I, _I, _P],
                    "zai_clamped_glu": [_P, _P, _I, _I, _I, _F, _F, _P],
                    "zai_act_mul": [_P, _P, _I, _I, _I, _I, _P],
+                   "zai_act_mul_rows": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
                    "zai_scale_softcap": [_P, ctypes.c_longlong, _F, _F, _P],
                    "zai_activation": [_P, _P, _I, _I, ctypes.c_longlong, _P],
                    "zai_weighted_sum": [_P, _P, _P, _I, _F, _F, ctypes.c_longlong, _P]},
@@ -112,6 +114,8 @@ _SIGNATURES = {
         "zai_skinny_gemm": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _P],
         "zai_skinny_gemm_clamped_glu": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _F, _F, _P],
         "zai_skinny_gemm_relu2": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _P],
+        "zai_skinny_gemm_added": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _P, _P, _P],
+        "zai_skinny_gemm_side": [_P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _P, _P],
         "zai_skinny_gemm_layernorm": [_P, _P, _P, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _F, _F, _P],
         "zai_skinny_conv": [_P, _P, _P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
         "zai_skinny_hint_next": [_P, ctypes.c_longlong],
@@ -428,10 +432,28 @@ def add_rmsnorm(h, delta, w, eps, out_dtype, delta_gamma=None, delta_eps=0.0):
 
 
 @_timed("norm")
-def add_cast(h, delta, out_dtype, delta_gamma=None, delta_eps=0.0):
+def add_rmsnorm_pair(h, delta, w_a, w_b, eps, out_dtype, delta_gamma=None, delta_eps=0.0):
+    """h += delta (as in `add_rmsnorm`), then two RMS norms of h, with weights w_a and w_b: what two sublayers side by side read."""
+    _cuda(h, delta, w_a, w_b, delta_gamma)
+    if h.dtype != torch.float32 or any(w is not None and w.dtype != torch.float32 for w in (w_a, w_b, delta_gamma)):
+        raise KernelError("the residual stream and norm weights are 32-bit")
+    if delta is not None and delta.dtype != out_dtype:
+        raise KernelError("the pending term should have the model's dtype")
+    N, H = h.shape
+    a, b = (torch.empty((N, H), dtype=out_dtype, device=h.device) for _ in range(2))
+    _check(_fn("norm", "zai_add_rmsnorm_pair")(_ptr(h), _ptr(delta), _ptr(delta_gamma), float(delta_eps), _ptr(w_a), _ptr(w_b), _ptr(a),
+                                               _ptr(b), _dt(a), float(eps), N, H, _stream()), "add_rmsnorm_pair")
+    return a, b
+
+
+@_timed("norm")
+def add_cast(h, delta, out_dtype, delta_gamma=None, delta_eps=0.0, delta2=None):
     """h += delta (in place, 32-bit; with `delta_gamma` the pending term passes an RMS norm with that weight first; nothing
-    with no delta), then h rounded to `out_dtype`: the input of a sublayer that reads the residual stream itself."""
-    _cuda(h, delta, delta_gamma)
+    with no delta) + `delta2` (a second term, added as it is), then h rounded to `out_dtype`: the input of a sublayer that
+    reads the residual stream itself."""
+    _cuda(h, delta, delta_gamma, delta2)
+    if delta2 is not None and (delta is None or delta2.dtype != out_dtype):
+        raise KernelError("a second pending term goes with a first one, both in the model's dtype")
     if h.dtype != torch.float32 or (delta_gamma is not None and delta_gamma.dtype != torch.float32):
         raise KernelError("the residual stream and norm weights are 32-bit")
     if delta is not None and delta.dtype != out_dtype:
@@ -439,7 +461,7 @@ def add_cast(h, delta, out_dtype, delta_gamma=None, delta_eps=0.0):
     N, H = h.shape
     out = torch.empty((N, H), dtype=out_dtype, device=h.device)
     _check(_fn("norm", "zai_add_normed_cast")(_ptr(h), _ptr(delta), _ptr(delta_gamma), float(delta_eps), _ptr(out), _dt(out), N, H,
-                                              _stream()), "add_cast")
+                                              _ptr(delta2), _stream()), "add_cast")
     return out
 
 
@@ -488,9 +510,10 @@ def _bias_through(w, beta):
 
 
 @_timed(_product_class)
-def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None):
+def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None, bias=None, addend=None):
     """The few-rows product kernel, if it takes these operands; else None.  `glu` = (limit, slope): the gated epilogue
-    with bounded branches instead of SiLU(gate) * up.  `plain_act="relu2"`: the square of relu as the bfloat16 epilogue."""
+    with bounded branches instead of SiLU(gate) * up.  `plain_act="relu2"`: the square of relu as the bfloat16 epilogue.
+    `bias` [O] (bfloat16) or, for 32-bit results, `addend` [M, O] (32-bit): added to the sums before they are rounded."""
     lazy = isinstance(x, LazyNorm)
     M = (x.rows.numel() if x.rows is not None else x.residual.data.shape[0]) if lazy else x.shape[0]
     O, K = w.shape
@@ -502,6 +525,12 @@ def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None):
         return None
     if plain_act is not None and lazy and getattr(x, "beta", None) is not None:
         return None
+    added = bias is not None or addend is not None
+    if added:
+        _cuda(bias, addend)
+        if (bias is not None and (bias.dtype != torch.bfloat16 or bias.numel() != O)) or (
+                addend is not None and (addend.dtype != torch.float32 or tuple(addend.shape) != (M, O))):
+            raise KernelError("a product's bias is bfloat16 [O], its addend 32-bit [M, O]")
     y = torch.empty((M, out_cols), dtype=out_dtype, device=w.device)
     _hint_next_weights(w)
     if plain_act is not None:
@@ -514,7 +543,12 @@ def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None):
         res = x.residual
         _cuda(res.data, x.delta, x.gamma, x.rows)
         h_out = torch.empty_like(res.data) if (x.rows is None and x.delta is not None) else None
-        if getattr(x, "beta", None) is not None:
+        if added:
+            beta_dot = _bias_through(w, x.beta) if getattr(x, "beta", None) is not None else None
+            _check(_fn("decode_gemm", "zai_skinny_gemm_added")(
+                _ptr(y), _ptr(w), None, _ptr(res.data), _ptr(x.delta), _ptr(x.gamma), _ptr(beta_dot), _ptr(x.rows), _ptr(h_out),
+                float(x.eps), M, O, K, epilogue, _ptr(bias), _ptr(addend), _stream()), "skinny_gemm")
+        elif getattr(x, "beta", None) is not None:
             # a layer norm: the kernel takes the mean off; the norm's bias goes through the product once per matrix
             limit, slope = (float(glu[0]), float(glu[1])) if glu is not None else (0.0, 1.0)
             _check(_fn("decode_gemm", "zai_skinny_gemm_layernorm")(
@@ -525,6 +559,10 @@ def _skinny(x, w, epilogue, out_cols, out_dtype, glu=None, plain_act=None):
                       float(x.eps), M, O, K, *tail), "skinny_gemm")
         if h_out is not None:
             res.data = h_out
+    elif added:
+        _cuda(x)
+        _check(_fn("decode_gemm", "zai_skinny_gemm_added")(_ptr(y), _ptr(w), _ptr(x), None, None, None, None, None, None, 0.0, M, O, K,
+                                                           epilogue, _ptr(bias), _ptr(addend), _stream()), "skinny_gemm")
     else:
         _cuda(x)
         _check(fn(_ptr(y), _ptr(w), _ptr(x), None, None, None, None, None, 0.0, M, O, K, *tail), "skinny_gemm")
@@ -626,10 +664,14 @@ def linear(x, w, out_dtype=None, bias=None):
     """x [N, K] times w [O, K] transposed.  x may be a LazyNorm.  Few rows in bfloat16 go to the
     fused few-rows kernel, many rows to the tcgen05 kernel where it is the faster one; a matrix kept
     in 32-bit is multiplied in 32-bit; the rest is the library's.  With `bias` [O] (in w's dtype) the
-    library's product adds it before the result is rounded."""
+    product adds it before the result is rounded."""
     in_dtype = x.dtype
     out_dtype = out_dtype or in_dtype
     if bias is not None:
+        if in_dtype == bias.dtype == torch.bfloat16 and out_dtype == torch.bfloat16:
+            y = _skinny(x, w, _EPI_BF16, w.shape[0], out_dtype, bias=bias)
+            if y is not None:
+                return y
         if isinstance(x, LazyNorm):
             x = x.materialize(sys.modules[__name__])
         return _library_product(x, w, out_dtype, bias)
@@ -647,6 +689,25 @@ def linear(x, w, out_dtype=None, bias=None):
         if y is not None:
             return y
     return _library_product(x, w, out_dtype)
+
+
+def linear_add(x, w, addend):
+    """x [N, K] times w [O, K] transposed, plus `addend` [N, O] in 32-bit; the sum is 32-bit."""
+    _cuda(addend)
+    if x.dtype == torch.bfloat16:
+        y = _skinny(x, w, _EPI_F32, w.shape[0], torch.float32, addend=addend)
+        if y is not None:
+            return y
+    return _library_sum(x, w, addend)
+
+
+@_timed("products")
+def _library_sum(x, w, addend):
+    if x.dtype == w.dtype == torch.bfloat16:
+        return torch.addmm(addend, x, w.t(), out_dtype=torch.float32)      # (sums in 32-bit from 16-bit operands)
+    if torch.backends.cuda.matmul.allow_tf32:
+        torch.backends.cuda.matmul.allow_tf32 = False
+    return torch.addmm(addend, x.float(), w.float().t())
 
 
 @_timed(lambda x, w, out_dtype, bias=None: "head" if out_dtype == torch.float32 and x.dtype != torch.float32 else "products")
@@ -1052,10 +1113,11 @@ def fused_decode_attention_available(dtype, heads, kv_heads, head_dim) -> bool:
 
 @_timed("attention (with q/k norm, rotation, page write)")
 def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_heads, head_dim, scale,
-                           window=None, write=True, q_map=0):
+                           window=None, write=True, q_map=0, scaling=None):
     """A decode step's attention in one kernel, from the qkv projection's rows [B, (Hq + 2 Hkv) D]:
     q/k RMSNorm, rotation, the new key and value into their page, attention over the pages in chunks
-    of keys, and the combination of the chunks.  Every row of the step is one token.  `q_map`: as in `qk_norm_rope`."""
+    of keys, and the combination of the chunks.  Every row of the step is one token.  `q_map`: as in `qk_norm_rope`;
+    `scaling`: of the rotation, as in `inverse_frequencies`."""
     _cuda(qkv, q_w, k_w)
     B, cols = qkv.shape
     if cols < ((heads // 2 if q_map else heads) + 2 * kv_heads) * head_dim:
@@ -1079,7 +1141,7 @@ def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, h
     if tickets is None or tickets.numel() < B * kv_heads:
         tickets = torch.zeros(max(B * kv_heads, 65536), dtype=torch.int32, device=dev)
         _tickets[str(dev)] = tickets
-    table = rope_table(step, rotary_dim, theta, dev) if rotary_dim else None
+    table = rope_table(step, rotary_dim, theta, dev, scaling) if rotary_dim else None
     bt = cache.block_table
     if USE_TMA_ATTENTION and _fn("attention_tma", "zai_decode_attention_tma_supports")(head_dim, heads, kv_heads, cache.page_size):
         _check(_fn("attention_tma", "zai_decode_attention_tma")(
@@ -1391,16 +1453,18 @@ def qkv_prepare(y, q_w, k_w, eps, scope, table, rot, step, cache, heads, kv_head
 
 
 @_timed("activation")
-def sigmoid_gate(o, gate, heads, head_dim, per_head):
+def sigmoid_gate(o, gate, heads, head_dim, per_head, row_dim=None):
     """o [N, heads * head_dim] times sigmoid(gate): gate [N, heads] (one number per head) or [N, heads * head_dim]; a
-    column slice is fine for the gate."""
+    column slice is fine for the gate.  `row_dim`: heads lie that far apart in o's rows (their values first, the rest is
+    passed over)."""
+    row_dim = head_dim if row_dim is None else int(row_dim)
     _cuda(o)
     gp, gs = _rows_view(gate)
     N = o.shape[0]
-    if gate.dtype != o.dtype or o.shape[1] != heads * head_dim or gate.shape[1] != (heads if per_head else heads * head_dim):
+    if gate.dtype != o.dtype or o.shape[1] != heads * row_dim or row_dim < head_dim or gate.shape[1] != (heads if per_head else heads * head_dim):
         raise KernelError("sigmoid_gate: operands do not fit together")
-    out = torch.empty_like(o)
-    _check(_fn("qkv_prepare", "zai_sigmoid_gate")(_ptr(out), _ptr(o), heads * head_dim, head_dim, gp, gs, _dt(o), int(bool(per_head)),
+    out = torch.empty((N, heads * head_dim), dtype=o.dtype, device=o.device)
+    _check(_fn("qkv_prepare", "zai_sigmoid_gate")(_ptr(out), _ptr(o), heads * row_dim, row_dim, gp, gs, _dt(o), int(bool(per_head)),
                                                   N, int(heads), int(head_dim), _stream()), "sigmoid_gate")
     return out
 
@@ -1538,7 +1602,8 @@ MOE_TALL_TILE_ROWS = 32      # from this many rows per expert on average, tiles 
 
 @_timed("experts")
 def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on="input", score="sigmoid", act="silu", limit=0.0,
-                   alpha=1.702, router_bias=None, unit=None, unit_gated=False):
+                   alpha=1.702, router_bias=None, unit=None, unit_gated=False, correction=None, groups=None, identities=0,
+                   weight_scale=1.0, onto=None):
     """A mixture of gated feed-forwards.  x [N, W]; w_router [E, W] 32-bit; w_gate_up [E, 2 F, W] (an expert's gate rows,
     then its up rows); w_down [E, W, F].  Every row goes to the `top` experts with the largest sigmoid(x . w_router^T)
     (32-bit); the scores are the weights (divided by their sum with `renorm`), applied to the expert's input or to its
@@ -1548,7 +1613,13 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
     `score="chosen"`: the logits themselves choose and the weights are the softmax over the chosen logits.  `router_bias` [E]
     32-bit is added to the logits (not with sigmoid scores).  `act="relu2"`: experts without a gate, down(relu(up)^2), w_gate_up
     being [E, F, W].  `unit` [N, W]: the rows of a feed-forward that every row passes, added in the same sum; with `unit_gated`
-    times sigmoid(x . w), w being the row of w_router [E + 1, W] behind the experts'."""
+    times sigmoid(x . w), w being the row of w_router [E + 1, W] behind the experts'.
+    `correction` [E + identities] 32-bit: the choice goes by score + correction (the weights by the score); `groups` = (count,
+    keep): the experts form `count` equal groups of neighbours and only those of the `keep` groups with the largest choice
+    values can be chosen; `identities`: that many rows of w_router behind the experts' stand for experts whose output is the
+    row itself; `weight_scale`: a factor on the weights.  (None of these with logit scores.)  `onto` = (h, other, cast): the
+    sum, with `other` [N, W] (rows of a mixer, or None), is added to the residual stream h [N, W] (in place, 32-bit) instead
+    of being returned; returns h rounded to x's dtype (None without `cast`)."""
     if score not in ("sigmoid", "softmax", "chosen") or act not in ("silu", "clamped", "relu2"):
         raise KernelError("routed_experts: score is sigmoid, softmax or chosen, act silu, clamped or relu2")
     gated = {"silu": 1, "clamped": 2, "relu2": 3}[act]
@@ -1557,21 +1628,30 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
     N, W = x.shape
     E, up_rows = w_gate_up.shape[0], w_gate_up.shape[1]
     F = up_rows if act == "relu2" else up_rows // 2
-    top = int(top)
+    top, E_all = int(top), E + int(identities)          # (identities count as experts for the router alone)
+    n_groups, keep = (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
+    _cuda(correction)
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E_all):
+        raise KernelError("routed_experts: the correction is one 32-bit number per expert and identity")
+    h, other, cast = onto if onto is not None else (None, None, True)
+    _cuda(h, other)
+    if h is not None and (h.dtype != torch.float32 or tuple(h.shape) != (N, W)) or (
+            other is not None and (other.dtype != x.dtype or tuple(other.shape) != (N, W))):
+        raise KernelError("routed_experts: the stream or the rows beside the experts do not fit")
     if unit_gated and unit is None or (unit is not None and (tuple(unit.shape) != (N, W) or unit.dtype != x.dtype)) or (
-            router_bias is not None and (router_bias.dtype != torch.float32 or router_bias.numel() != E or score == "sigmoid")):
+            router_bias is not None and (router_bias.dtype != torch.float32 or router_bias.numel() != E_all or score == "sigmoid")):
         raise KernelError("routed_experts: the router's bias or the unit's rows do not fit")
-    if (w_router.dtype != torch.float32 or tuple(w_router.shape) != (E + int(unit_gated), W) or up_rows != (F if act == "relu2" else 2 * F)
+    if (w_router.dtype != torch.float32 or tuple(w_router.shape) != (E_all + int(unit_gated), W) or up_rows != (F if act == "relu2" else 2 * F)
             or w_gate_up.shape[2] != W or tuple(w_down.shape) != (E, W, F) or w_gate_up.dtype != x.dtype or w_down.dtype != x.dtype
             or weight_on not in ("input", "output")):
         raise KernelError("routed_experts: operands do not fit together")
     dev, dt, lib = x.device, _dt(x), "moe"
-    out = torch.empty((N, W), dtype=x.dtype, device=dev)
+    out = torch.empty((N, W), dtype=x.dtype, device=dev) if cast else None
     if N == 0:
         return out
-    tall = dt == _BF16 and W % 8 == 0 and F % 8 == 0 and N * top >= MOE_TALL_TILE_ROWS * E
+    tall = dt == _BF16 and W % 8 == 0 and F % 8 == 0 and N * top >= MOE_TALL_TILE_ROWS * E_all
     # many rows an expert: tiles of 128 rows and both products on the 5th-generation tensor cores (grouped tcgen05)
-    grouped = (tall and USE_MOE_GROUPED_TC and N * top >= MOE_GROUPED_TILE_ROWS * E
+    grouped = (tall and USE_MOE_GROUPED_TC and N * top >= MOE_GROUPED_TILE_ROWS * E_all
                and _fn("gemm_tc", "zai_gemm_tc_supports")(128, up_rows, W, _EPI_SWIGLU if act == "silu" else _EPI_BF16)
                and _fn("gemm_tc", "zai_gemm_tc_supports")(128, W, F, _EPI_F32))
     TM = 128 if grouped else 64 if tall else 16
@@ -1584,15 +1664,22 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
     counts, tile_expert = meta[4 * N * top:4 * N * top + E], meta[4 * N * top + E:4 * N * top + E + max_tiles]
     unit_gate = meta[4 * N * top + E + max_tiles:].view(torch.float32) if unit_gated else None
     on_input = int(weight_on == "input")
-    _check(_fn(lib, "zai_moe_route")(_ptr(ids), _ptr(wts), _ptr(rank), _ptr(counts), xp, xs, dt, _ptr(w_router), N, W, E, top,
+    _check(_fn(lib, "zai_moe_route")(_ptr(ids), _ptr(wts), _ptr(rank), _ptr(counts), xp, xs, dt, _ptr(w_router), N, W, E_all, top,
                                      int(bool(renorm)), {"sigmoid": 0, "softmax": 1, "chosen": 2}[score], _ptr(router_bias),
-                                     _ptr(unit_gate), _stream()), "moe_route")
+                                     _ptr(unit_gate), _ptr(correction), n_groups, keep, E, float(weight_scale), _stream()), "moe_route")
     rows = max_tiles * TM
     x_sorted = torch.empty((rows, W), dtype=x.dtype, device=dev)
     _check(_fn(lib, "zai_moe_gather")(_ptr(x_sorted), _ptr(dest), _ptr(tile_expert), xp, xs, dt, _ptr(ids), _ptr(wts), _ptr(rank),
                                       _ptr(counts), N, W, E, top, TM, max_tiles, on_input, _stream()), "moe_gather")
     hidden = torch.empty((rows, F), dtype=x.dtype, device=dev)
     y = torch.empty((rows, W), dtype=torch.float32, device=dev)
+
+    def combine():
+        _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _ptr(unit), _ptr(unit_gate),
+                                           xp if identities else None, xs if identities else 0, _ptr(h), _ptr(other), _stream()),
+               "moe_combine")
+        return out
+
     if grouped:
         tc = _fn("gemm_tc", "zai_gemm_tc_grouped")
         if gated == 2:        # the plain grouped product, then the bounded activation on its gate|up rows
@@ -1606,18 +1693,12 @@ def routed_experts(x, w_router, w_gate_up, w_down, top, renorm=False, weight_on=
         _check(tc(_ptr(y), _ptr(w_down), _ptr(hidden), _ptr(tile_expert), _status_ptr(dev), max_tiles, E, W, F,
                   _EPI_F32_PAIR if USE_MOE_DOWN_PAIR else _EPI_F32, _stream()),
                "gemm_tc_grouped (down)")
-        _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _ptr(unit),
-                                               _ptr(unit_gate), _stream()),
-               "moe_combine")
-        return out
+        return combine()
     _check(_fn(lib, "zai_moe_gemm")(_ptr(hidden), int(dt == _F32), _ptr(x_sorted), _ptr(w_gate_up), dt, _ptr(tile_expert), max_tiles,
                                     TM, W, F, gated, float(limit), float(alpha), _stream()), "moe_gemm (gate/up)")
     _check(_fn(lib, "zai_moe_gemm")(_ptr(y), 1, _ptr(hidden), _ptr(w_down), dt, _ptr(tile_expert), max_tiles, TM, F, W, 0, 0.0, 0.0,
                                     _stream()), "moe_gemm (down)")
-    _check(_fn(lib, "zai_moe_combine")(_ptr(out), dt, _ptr(y), _ptr(dest), _ptr(wts), N, W, top, 1 - on_input, _ptr(unit),
-                                               _ptr(unit_gate), _stream()),
-           "moe_combine")
-    return out
+    return combine()
 
 
 # ----------------------------------------------------------------------------- gated feed-forward with any activation, mLSTM
@@ -1645,6 +1726,38 @@ def linear_glu(x, w_gate_up, ff_dim, kind):
         if y is not None:
             return y
     return act_mul(linear(x, w_gate_up), ff_dim, kind)
+
+
+def linear_side(x, w, table, ids, at):
+    """gelu_tanh(x . w^T) times the rows' entries at .. at + O - 1 of `table` [rows, columns] by token id: x [N, K], w [O, K].  Few
+    rows in bfloat16: the product's epilogue; else a kernel behind the product."""
+    _cuda(w, table, ids)
+    N, (O, K), (rows, ld), at = x.shape[0], w.shape, table.shape, int(at)
+    if ids.numel() != N or ids.dtype != torch.int32 or table.dtype != x.dtype or at < 0 or at + O > ld:
+        raise KernelError("linear_side: the table's entries do not fit the product")
+    if x.dtype == torch.bfloat16 and x.is_contiguous() and _fn("decode_gemm", "zai_skinny_gemm_supports")(N, O, K, _EPI_BF16, 0):
+        return _skinny_side(x, w, table, ids, at)
+    y = linear(x, w)
+    return _act_mul_rows(y, table, ids, at)
+
+
+@_timed("products")
+def _skinny_side(x, w, table, ids, at):
+    N, (O, K) = x.shape[0], w.shape
+    y = torch.empty((N, O), dtype=x.dtype, device=x.device)
+    _hint_next_weights(w)
+    _check(_fn("decode_gemm", "zai_skinny_gemm_side")(_ptr(y), _ptr(w), _ptr(x), N, O, K, _ptr(table), _ptr(ids), table.shape[0], table.shape[1],
+                                                      at, _status_ptr(x.device), _stream()), "skinny_gemm_side")
+    return y
+
+
+@_timed("activation")
+def _act_mul_rows(y, table, ids, at):
+    out = torch.empty_like(y)
+    _check(_fn("activation", "zai_act_mul_rows")(_ptr(out), _ptr(y), _ptr(table), _ptr(ids), table.shape[0], table.shape[1], at, _dt(y),
+                                                 y.shape[0], y.shape[1], _ACT_KINDS["gelu_tanh"], _status_ptr(y.device), _stream()),
+           "act_mul_rows")
+    return out
 
 
 @_timed("attention")

@@ -24,6 +24,8 @@ class Model:
         self.blocks = [make_block(ls) for ls in spec.layers]
         self.final_norm = make_part("norm", spec.final_norm)
         self.head = make_part("head", spec.head, **sizes)
+        self.tables = {name: make_part("table", t, vocab=spec.vocab_size) for name, t in spec.tables.items()}
+        self.keeps_embedding = any(getattr(b, "reads_embedding", False) for b in self.blocks)
         for k, call in enumerate(spec.order):
             if not 0 <= call.layer < len(self.blocks):
                 raise ValueError(f"order[{k}] names layer {call.layer}, but there are {len(self.blocks)} layers")
@@ -42,7 +44,7 @@ class Model:
         out = [("", self.embedding)]
         for ls, block in zip(self.spec.layers, self.blocks):
             out += [(ls.prefix, part) for part in [block] + list(block.parts().values())]
-        return out + [("", self.final_norm), ("", self.head)]
+        return out + [("", self.final_norm), ("", self.head)] + [("", t) for t in self.tables.values()]
 
     def all_parts(self) -> List:
         return [part for _, part in self._owners()]
@@ -64,6 +66,9 @@ class Model:
                 part.bind({local: tensors[prefix + local] for local in names}, dtype)
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding)
+        for part in self.all_parts():
+            if hasattr(part, "attach"):
+                part.attach(self.tables)
 
     # ------------------------------------------------------------------ cache needs
     def cache_needs(self) -> List:
@@ -93,6 +98,8 @@ class Model:
     def _forward(self, step, cache, ops) -> torch.Tensor:
         step.scratch.clear()                # per-step tables are computed anew (also inside a graph capture)
         h = Residual(self.embedding.forward(step.token_ids, step))
+        if self.keeps_embedding:            # a copy in the activations' dtype: the stream itself is added to in place
+            step.scratch["embedding"] = ops.add_cast(h.data, None, step.dtype)
         pending = None
         for k, call in enumerate(self.spec.order):
             h, pending = self.blocks[call.layer].forward(h, pending, step, cache.views(k, step), call.cache_of is None)

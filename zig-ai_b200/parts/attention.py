@@ -18,7 +18,7 @@ Further options, for designs that have them: `bias` (q, k and v projections with
 before the split into heads); `chunk` (a query sees back to the start of its chunk of that many positions,
 counted from position 0 of the request: j <= i and j // chunk == i // chunk); `gate="head"` (a fourth
 projection of one number per query head; a head's output is multiplied by its sigmoid before the output
-projection); a position part that pairs dimensions (2i, 2i+1) or stretches its frequencies.  With any of them
+projection); `out_bias` (a bias on the output projection, with `bias`); a position part that pairs dimensions (2i, 2i+1) or stretches its frequencies.  With any of them
 the projections run as one product q|k|v|gate and one kernel norms, rotates and writes the pages
 (`ops.qkv_prepare`); an interleaved pairing is turned into the half-split one by reordering the rows of the q
 and k projections (with their biases and norm weights) at load.
@@ -58,7 +58,7 @@ import math
 
 import torch
 
-from .base import Mixer, PagedKVNeed, ParamDecl, make_part, register_part, PartSpec
+from .base import Mixer, PagedKVNeed, ParamDecl, make_part, register_part, PartSpec, stack_rows
 
 
 class Attention(Mixer):
@@ -69,7 +69,8 @@ class Attention(Mixer):
     def __init__(self, hidden: int, heads: int, kv_heads: int, head_dim: int, qk_norm: bool, eps: float,
                  position: PartSpec, window=None, scale=None, kv_proj: bool = True, value_dim=None,
                  value_norm: bool = False, names=None, bias: bool = False, norm_scope: str = "head", chunk=None, gate=None,
-                 q_temp=None, softcap=None, rel_bias=None, sink: bool = False, keep_first: int = 0, v_mix=None, differential=None):
+                 q_temp=None, softcap=None, rel_bias=None, sink: bool = False, keep_first: int = 0, v_mix=None, differential=None,
+                 out_bias: bool = False):
         self.differential = None if differential is None else float(differential["diff"])
         if self.differential is not None:
             # to everything below, a head is a pair of query heads over keys of twice the size
@@ -93,10 +94,12 @@ class Attention(Mixer):
         self.cache_dim = max(self.head_dim, self.value_dim)      # the head size of the pages and the kernels
         self.names = {"q": "attn_q.weight", "k": "attn_k.weight", "v": "attn_v.weight", "o": "attn_output.weight",
                       "q_norm": "attn_q_norm.weight", "k_norm": "attn_k_norm.weight", "q_bias": "attn_q.bias",
-                      "k_bias": "attn_k.bias", "v_bias": "attn_v.bias", "g": "attn_gate.weight", "rel": "attn_rel_bias",
+                      "k_bias": "attn_k.bias", "v_bias": "attn_v.bias", "o_bias": "attn_output.bias", "g": "attn_gate.weight", "rel": "attn_rel_bias",
                       "sink": "attn_sink", "vmix": "attn_vmix", "lq1": "attn_lambda_q1", "lk1": "attn_lambda_k1",
                       "lq2": "attn_lambda_q2", "lk2": "attn_lambda_k2", **(names or {})}
-        self.bias, self.norm_scope, self.gate = bool(bias), str(norm_scope), gate
+        self.bias, self.norm_scope, self.gate, self.out_bias = bool(bias), str(norm_scope), gate, bool(out_bias)
+        if self.out_bias and not self.bias:
+            raise ValueError("a bias on the output projection goes with biases on the others")
         self.chunk = None if chunk is None else int(chunk)
         if self.norm_scope not in ("head", "whole") or self.gate not in (None, "head"):
             raise ValueError("norm_scope is 'head' or 'whole'; gate is None or 'head'")
@@ -120,6 +123,11 @@ class Attention(Mixer):
                              or self.shaped or self.q_temp or self.v_mix
                              or getattr(self.position, "pairing", "half_split") != "half_split"
                              or getattr(self.position, "scaling", None) is not None)
+        # what the kernel that does a single token's whole attention serves beside them: plain windowed scores, norms per head,
+        # keys at least as wide as the values
+        self.one_kernel_decode = bool(self.prepared and not self.shaped and not self.q_temp and not self.v_mix and self.chunk is None
+                                      and self.norm_scope == "head" and self.value_dim <= self.head_dim
+                                      and self.position.rotation() is not None)
         if self.prepared and (self.value_norm or not self.kv_proj):
             raise ValueError("value_norm and a borrowed cache are not combined with bias, whole norm, chunk or gate")
         if self.prepared:
@@ -149,6 +157,8 @@ class Attention(Mixer):
             p[nm["q_bias"]] = ParamDecl((q_dim,), "vector", init="conv")
             p[nm["k_bias"]] = ParamDecl((kv_dim,), "vector", init="conv")
             p[nm["v_bias"]] = ParamDecl((self.kv_heads * self.value_dim,), "vector", init="conv")
+        if self.out_bias:
+            p[nm["o_bias"]] = ParamDecl((self.hidden,), "vector", init="conv")
         if self.gate:
             p[nm["g"]] = ParamDecl((self.heads, self.hidden))
         if self.rel_bias:
@@ -190,14 +200,26 @@ class Attention(Mixer):
             return t.reshape((n_heads, D) + tuple(t.shape[1:])).index_select(1, idx).reshape(t.shape).contiguous()
 
         q, k, v = heads_reordered(tensors[nm["q"]], H), heads_reordered(tensors[nm["k"]], G), tensors[nm["v"]]
-        mats = [q, k, v] + ([tensors[nm["g"]]] if self.gate else [])
-        self.w_qkv = torch.cat(mats, dim=0).contiguous()
-        self.b_qkv = None
+        b = None
         if self.bias:
             b = [heads_reordered(tensors[nm["q_bias"]], H), heads_reordered(tensors[nm["k_bias"]], G), tensors[nm["v_bias"]]]
-            if self.gate:
-                b.append(b[0].new_zeros(H))
+        self.y_value_dim = Dv                      # the values' size in the projection's rows
+        if self.one_kernel_decode and Dv < D:
+            # rows of zeros make the values as wide as the keys, so that the kernel for single tokens reads them as they are
+            wide = lambda t: torch.cat([t.reshape((G, Dv) + tuple(t.shape[1:])), t.new_zeros((G, D - Dv) + tuple(t.shape[1:]))],
+                                       dim=1).reshape((G * D,) + tuple(t.shape[1:]))
+            v = wide(v)
+            if b is not None:
+                b[2] = wide(b[2])
+            self.y_value_dim = D
+        mats = [q, k, v] + ([tensors[nm["g"]]] if self.gate else [])
+        self.w_qkv, _ = stack_rows([torch.cat(mats, dim=0)])        # (rows of the product on 16-byte boundaries)
+        self.b_qkv = self.b_o = None
+        if self.bias:
+            b += [b[0].new_zeros(self.w_qkv.shape[0] - sum(t.shape[0] for t in b))]
             self.b_qkv = torch.cat(b).to(self.w_qkv.dtype).contiguous()
+        if self.out_bias:
+            self.b_o = tensors[nm["o_bias"]].to(self.w_qkv.dtype).contiguous()
         self.q_norm, self.k_norm = tensors.get(nm["q_norm"]), tensors.get(nm["k_norm"])
         if self.norm_scope == "whole":
             self.q_norm, self.k_norm = heads_reordered(self.q_norm, H), heads_reordered(self.k_norm, G)
@@ -205,10 +227,10 @@ class Attention(Mixer):
             self.q_norm, self.k_norm = self.q_norm[idx].contiguous(), self.k_norm[idx].contiguous()
         self.norm_eps = self.eps
         self.w_o = tensors[nm["o"]]
-        if Dp != Dv:
+        if Dp != Dv and not self.gate:             # (the gate's kernel leaves the zeros behind a head's values out)
             w = self.w_o.reshape(self.hidden, H, Dv)
             self.w_o = torch.cat([w, w.new_zeros(self.hidden, H, Dp - Dv)], dim=2).reshape(self.hidden, -1).contiguous()
-        self.gate_at = H * D + G * D + G * Dv
+        self.gate_at = H * D + G * D + G * self.y_value_dim
         self.v_at = H * D + G * D
         self.bias_table = self.distance_table(tensors[nm["rel"]]) if self.rel_bias else None
         self.sink_w = tensors[nm["sink"]].float().contiguous() if self.sink else None
@@ -218,6 +240,13 @@ class Attention(Mixer):
     def _forward_prepared(self, x, step, cache, write_cache):
         ops, H, G, D, Dv, Dp = step.ops, self.heads, self.kv_heads, self.head_dim, self.value_dim, self.cache_dim
         y = ops.linear(x, self.w_qkv, bias=self.b_qkv)
+        fused = getattr(ops, "fused_decode_attention_available", None)
+        if self.one_kernel_decode and step.decode_only and fused is not None and fused(y.dtype, H, G, Dp):
+            # norm, rotation, page write, attention and the combination of the key ranges in one kernel
+            rot = self.position.rotation()
+            o = ops.decode_attention_fused(y, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache, H, G, Dp, self.scale,
+                                           self.window, write_cache, scaling=rot[2])
+            return self._prepared_output(o, y, ops)
         dims, table = self.position.table(step, y.device)
         scope = 0 if not self.qk_norm else (2 if self.norm_scope == "whole" else 1)
         more = {}
@@ -229,16 +258,19 @@ class Attention(Mixer):
             if "attention.v_first" not in step.scratch:
                 raise RuntimeError("a layer mixes its values with an earlier layer's, and no earlier layer has left any")
             more.update(v_first=step.scratch["attention.v_first"], v_lambda=self.v_lambda)
-        q = ops.qkv_prepare(y, self.q_norm, self.k_norm, self.norm_eps, scope, table, dims, step, cache, H, G, D, Dv, Dp,
+        q = ops.qkv_prepare(y, self.q_norm, self.k_norm, self.norm_eps, scope, table, dims, step, cache, H, G, D, self.y_value_dim, Dp,
                             write_cache, **more)
         if self.shaped:
             o = ops.paged_attention(q, step, cache, H, G, Dp, self.scale, self.window, softcap=self.softcap, bias=self.bias_table,
                                     sink=self.sink_w, keep_first=self.keep_first)
         else:
             o = ops.paged_attention(q, step, cache, H, G, Dp, self.scale, self.window, chunk=self.chunk)
+        return self._prepared_output(o, y, ops)
+
+    def _prepared_output(self, o, y, ops):
         if self.gate:
-            o = ops.sigmoid_gate(o, y[:, self.gate_at:self.gate_at + H], H, Dp, True)
-        return ops.linear(o, self.w_o)
+            o = ops.sigmoid_gate(o, y[:, self.gate_at:self.gate_at + self.heads], self.heads, self.value_dim, True, row_dim=self.cache_dim)
+        return ops.linear(o, self.w_o, bias=self.b_o)
 
     def bind(self, tensors, dtype):
         if self.prepared:

@@ -62,6 +62,7 @@ class ModelSpec:
     order: List[LayerCall]
     final_norm: PartSpec
     head: PartSpec
+    tables: Dict[str, PartSpec] = field(default_factory=dict)     # tables by token id that several layers read (family table)
 
 
 # --------------------------------------------------------------------------- tensors a part owns
@@ -232,6 +233,24 @@ class FeedForward(Part):
     def forward(self, x, step):
         raise NotImplementedError
 
+    def forward_onto(self, x, step, h, other, cast=True):
+        """Add forward(x) and `other` [N, hidden] (a mixer's output) to the residual stream `h`, in 32-bit; returns the stream
+        in the activations' dtype (None without `cast`).  A part whose last kernel can do the addition overrides this."""
+        out = step.ops.add_cast(h.data, other, step.dtype, delta2=self.forward(x, step))
+        return out if cast else None
+
+
+class TokenInput(Part):
+    """A term that depends on the stream and on the token itself, added behind a layer's sublayers: forward(x, step) -> a
+    `NormedTerm` (or a plain pending term); x [N, hidden] is the stream in the activations' dtype.  `attach(tables)` hands it
+    the model's tables (`ModelSpec.tables`, parts by name) after all tensors are bound."""
+
+    def attach(self, tables) -> None:
+        pass
+
+    def forward(self, x, step):
+        raise NotImplementedError
+
 
 class Norm(Part):
     """forward(h, delta or None, step) -> normed [N, hidden] in the model's dtype.  `h` is the
@@ -248,6 +267,10 @@ class PositionEncoding(Part):
     (rotary_dim, theta)), or transforms q and k itself in `apply`."""
 
     def rotary(self) -> Optional[Tuple[int, float]]:
+        return None
+
+    def rotation(self):
+        """(rotary_dim, theta, scaling) if this is a rotation of the first dimensions from a table, else None."""
         return None
 
     def apply(self, q, k, positions, step):
@@ -331,13 +354,14 @@ class Head(Part):
 
 # --------------------------------------------------------------------------- registries of parts
 _REGISTRIES: Dict[str, Dict[str, Callable]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "embedding": {}, "head": {},
+    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "block": {}, "embedding": {}, "head": {}, "table": {},
+    "token_input": {},
 }
 
 
 def register_part(family: str, kind: str, factory: Callable, replace: bool = False) -> None:
     """Make a part available under `kind` in one of the families mixer, feed_forward, norm,
-    position, block, embedding, head.  `factory(**params)` returns the part."""
+    position, block, embedding, head, table, token_input.  `factory(**params)` returns the part."""
     reg = _REGISTRIES[family]
     if kind in reg and not replace:
         raise ValueError(f"{family} '{kind}' is already registered")

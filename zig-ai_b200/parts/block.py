@@ -9,7 +9,7 @@ pending term into the next norm's kernel, which adds it into the 32-bit residual
 """
 from __future__ import annotations
 
-from .base import Block, NormedTerm, register_part
+from .base import Block, NormedTerm, ParamDecl, register_part
 
 
 class PreNormResidual(Block):
@@ -118,6 +118,81 @@ class PostNormResidual(Block):
         return h, self._term(f, self.ff_norm)
 
 
+class ParallelResidual(Block):
+    """Two sublayers side by side, each behind a norm of its own of the same stream, then optionally a term from the token:
+
+        h = h + (mixer(norm_a(h)) + feed_forward(norm_b(h)));   h = h + token_input(h)
+
+    Both norms are one kernel (which also adds what is pending); the feed-forward's last kernel adds its own and the mixer's
+    output to the stream and rounds it for the token input, whose normed term travels on to whatever comes next."""
+    graph_safe = True      # forward launches kernels only; nothing is read back to the host
+
+    def __init__(self, mixer, mixer_norm, feed_forward=None, ff_norm=None, token_input=None):
+        super().__init__()
+        self.mixer_norm = self.sub("mixer_norm", "norm", mixer_norm)
+        self.mixer = self.sub("mixer", "mixer", mixer)
+        self.feed_forward = self.token_input = None
+        if feed_forward is not None:
+            self.ff_norm = self.sub("ff_norm", "norm", ff_norm)
+            self.feed_forward = self.sub("feed_forward", "feed_forward", feed_forward)
+        if token_input is not None:
+            self.token_input = self.sub("token_input", "token_input", token_input)
+
+    def params(self):
+        return {}
+
+    def forward(self, h, pending, step, cache, write_cache=True):
+        if self.feed_forward is None:
+            r = self.mixer_norm.forward(h, pending, step, lazy=self.mixer.accepts_lazy_input)
+            pending = self.mixer.forward(r, step, self.cache_for(self.mixer, cache), write_cache)
+            if self.token_input is None:
+                return h, pending
+            x = step.ops.add_cast(h.data, pending, step.dtype)
+        else:
+            ra, rb = self.mixer_norm.forward_pair(h, pending, step, self.ff_norm)
+            m = self.mixer.forward(ra, step, self.cache_for(self.mixer, cache), write_cache)
+            x = self.feed_forward.forward_onto(rb, step, h, m, cast=self.token_input is not None)
+            if self.token_input is None:
+                return h, None
+        return h, self.token_input.forward(x, step)
+
+
+class StreamMerge(Block):
+    """A step of the running order with no sublayers: the stream is replaced by a product of itself and the embedding's output,
+
+        h <- W [h; h0] = W_a h + W_b h0
+
+    (ahead of every pass of layers that run several times, for instance).  The second product is the same wherever the step
+    stands in the order: it is made at the first one and kept, in 32-bit, for the rest of the forward pass."""
+    graph_safe = True
+    reads_embedding = True     # the model keeps the embedding's output, in the activations' dtype, in step.scratch["embedding"]
+
+    def __init__(self, hidden: int, weight: str):
+        super().__init__()
+        self.hidden, self.weight_name = int(hidden), weight
+
+    def params(self):
+        return {self.weight_name: ParamDecl((self.hidden, 2 * self.hidden))}
+
+    def bind(self, tensors, dtype):
+        w = tensors[self.weight_name]
+        self.w_stream, self.w_embedding = w[:, :self.hidden].contiguous(), w[:, self.hidden:].contiguous()
+
+    def forward(self, h, pending, step, cache, write_cache=True):
+        import torch
+        ops, key = step.ops, ("stream_merge", id(self))
+        if key not in step.scratch:
+            step.scratch[key] = ops.linear(step.scratch["embedding"], self.w_embedding, out_dtype=torch.float32)
+        if isinstance(pending, NormedTerm):
+            x = ops.add_cast(h.data, pending.data, step.dtype, pending.gamma, pending.eps)
+        else:
+            x = ops.add_cast(h.data, pending, step.dtype)
+        h.data = ops.linear_add(x, self.w_stream, step.scratch[key])
+        return h, None
+
+
+register_part("block", "parallel_residual", ParallelResidual)
+register_part("block", "stream_merge", StreamMerge)
 register_part("block", "prenorm_residual", PreNormResidual)
 register_part("block", "postnorm_residual", PostNormResidual)
 register_part("block", "sandwich_residual", SandwichResidual)

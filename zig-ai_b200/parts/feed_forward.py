@@ -119,18 +119,34 @@ class RoutedExperts(FeedForward):
     `score="chosen"`: the logits choose and the weights are the softmax over the chosen logits alone; `router_bias` adds a
     learned number per expert (name "router_bias") to the logits.  `expert_act="relu2"`: experts without a gate,
     down_e( relu(up_e(x))^2 ).  `shared_gate`: the shared feed-forward's output times sigmoid(x . w) with a learned row w (name
-    "shared_gate"), computed in 32-bit with the router."""
+    "shared_gate"), computed in 32-bit with the router.
+
+    Options of the choice (with sigmoid or softmax scores): `correction` (a learned number per expert, name "correction", is
+    added to the scores for the choice alone); `groups` = {count, keep} (equal groups of neighbouring experts; only the experts
+    of the `keep` groups with the largest choice values can be chosen); `identities` (that many further outputs of the router
+    stand for experts without tensors whose output is x itself); `weight_scale` (a factor on the weights)."""
     accepts_lazy_input = False    # the router and the experts read the normed rows themselves
     graph_safe = True             # routing stays on the device: forward launches kernels only
     kernel_libs = ("moe", "gemm_tc")      # (gemm_tc: the grouped products of steps with many rows an expert, bfloat16)
 
     def __init__(self, hidden: int, ff_dim: int, experts: int, top: int, renormalize: bool = False, weight_on: str = "input",
                  names=None, score: str = "sigmoid", expert_act: str = "silu", limit: float = 0.0, alpha: float = 1.702, shared=None,
-                 router_bias: bool = False, shared_gate: bool = False):
+                 router_bias: bool = False, shared_gate: bool = False, correction: bool = False, groups=None, identities: int = 0,
+                 weight_scale: float = 1.0):
         self.hidden, self.ff_dim, self.experts, self.top = int(hidden), int(ff_dim), int(experts), int(top)
         self.renormalize, self.weight_on = bool(renormalize), weight_on
-        if not 1 <= self.top <= self.experts or self.top > 32:
-            raise ValueError(f"a token uses between 1 and min(experts, 32) experts, not {self.top} of {self.experts}")
+        self.correction, self.identities, self.weight_scale = bool(correction), int(identities), float(weight_scale)
+        self.outputs = self.experts + self.identities                # what the router scores
+        self.groups = None if groups is None else (int(groups["count"]), int(groups["keep"]))
+        if not 1 <= self.top <= self.outputs or self.top > 32:
+            raise ValueError(f"a token uses between 1 and min(experts, 32) experts, not {self.top} of {self.outputs}")
+        if self.groups is not None:
+            count, keep = self.groups
+            if count < 1 or self.outputs % count or not 1 <= keep <= count or keep * (self.outputs // count) < self.top:
+                raise ValueError("the experts form equal groups, and the kept groups hold enough of them")
+        self.chosen_apart = bool(self.correction or self.groups or self.identities or self.weight_scale != 1.0)
+        if self.chosen_apart and score == "chosen":
+            raise ValueError("a correction, groups, identities and a weight factor go with sigmoid or softmax scores")
         if weight_on not in ("input", "output"):
             raise ValueError("weight_on is 'input' or 'output'")
         if score not in ("sigmoid", "softmax", "chosen") or expert_act not in ("silu", "clamped", "relu2"):
@@ -144,13 +160,16 @@ class RoutedExperts(FeedForward):
         self.shared = None if shared is None else make_part("feed_forward", shared)
         if self.shared is not None:
             self.kernel_libs = type(self).kernel_libs + tuple(getattr(self.shared, "kernel_libs", ()))
-        self.names = {"router": "ffn_router.weight", "router_bias": "ffn_router.bias", "shared_gate": "ffn_shared_gate.weight", "gate": "ffn_gate.{e}.weight", "up": "ffn_up.{e}.weight",
+        self.names = {"router": "ffn_router.weight", "router_bias": "ffn_router.bias", "correction": "ffn_router.correction",
+                      "shared_gate": "ffn_shared_gate.weight", "gate": "ffn_gate.{e}.weight", "up": "ffn_up.{e}.weight",
                       "down": "ffn_down.{e}.weight", **(names or {})}
 
     def params(self):
-        nm, p = self.names, {self.names["router"]: ParamDecl((self.experts, self.hidden), "vector", init="conv")}
+        nm, p = self.names, {self.names["router"]: ParamDecl((self.outputs, self.hidden), "vector", init="conv")}
         if self.router_bias:
-            p[nm["router_bias"]] = ParamDecl((self.experts,), "vector", init="conv")
+            p[nm["router_bias"]] = ParamDecl((self.outputs,), "vector", init="conv")
+        if self.correction:
+            p[nm["correction"]] = ParamDecl((self.outputs,), "vector", init="conv")
         if self.shared_gate:
             p[nm["shared_gate"]] = ParamDecl((1, self.hidden), "vector", init="conv")
         for e in range(self.experts):
@@ -171,6 +190,7 @@ class RoutedExperts(FeedForward):
             self.w_router = torch.cat([self.w_router, tensors[nm["shared_gate"]].float().reshape(1, self.hidden)], dim=0)
         self.w_router = self.w_router.contiguous()
         self.b_router = tensors[nm["router_bias"]].float().contiguous() if self.router_bias else None
+        self.w_correction = tensors[nm["correction"]].float().contiguous() if self.correction else None
         if self.expert_act == "relu2":
             self.w_gate_up = torch.stack([tensors[nm["up"].format(e=e)] for e in E]).contiguous()  # [E, F, hidden]
         else:
@@ -179,14 +199,22 @@ class RoutedExperts(FeedForward):
         self.w_down = torch.stack([tensors[nm["down"].format(e=e)] for e in E]).contiguous()   # [E, hidden, F]
         self.dtype = dtype
 
+    def _routed(self, x, step, unit, onto=None):
+        """The experts' sum with the shared feed-forward's rows in it."""
+        more = {}
+        if self.chosen_apart:
+            more = dict(correction=self.w_correction, groups=self.groups, identities=self.identities, weight_scale=self.weight_scale)
+        if onto is not None:
+            more["onto"] = onto
+        return step.ops.routed_experts(x, self.w_router, self.w_gate_up, self.w_down, self.top, self.renormalize, self.weight_on,
+                                       score=self.score, act=self.expert_act, limit=self.limit, alpha=self.alpha,
+                                       router_bias=self.b_router, unit=unit, unit_gated=self.shared_gate, **more)
+
     def forward(self, x, step):
         ops = step.ops
-        if self.score == "chosen" or self.expert_act == "relu2" or self.router_bias or self.shared_gate:
+        if self.score == "chosen" or self.expert_act == "relu2" or self.router_bias or self.shared_gate or self.chosen_apart:
             # the shared feed-forward's rows join in the sum over the chosen experts
-            unit = None if self.shared is None else self.shared.forward(x, step)
-            return ops.routed_experts(x, self.w_router, self.w_gate_up, self.w_down, self.top, self.renormalize, self.weight_on,
-                                      score=self.score, act=self.expert_act, limit=self.limit, alpha=self.alpha,
-                                      router_bias=self.b_router, unit=unit, unit_gated=self.shared_gate)
+            return self._routed(x, step, None if self.shared is None else self.shared.forward(x, step))
         if self.score == "sigmoid" and self.expert_act == "silu":
             y = ops.routed_experts(x, self.w_router, self.w_gate_up, self.w_down, self.top, self.renormalize, self.weight_on)
         else:
@@ -195,6 +223,10 @@ class RoutedExperts(FeedForward):
         if self.shared is None:
             return y
         return ops.weighted_sum(y, self.shared.forward(x, step), 1.0, 1.0)
+
+    def forward_onto(self, x, step, h, other, cast=True):
+        """The combine adds the experts' sum and `other` to the residual stream itself."""
+        return self._routed(x, step, None if self.shared is None else self.shared.forward(x, step), onto=(h.data, other, cast))
 
 
 register_part("feed_forward", "swiglu", SwiGlu)

@@ -43,6 +43,17 @@ class RmsNorm(Norm):
         return x.materialize(step.ops)
 
 
+    def forward_pair(self, h, delta, step, other):
+        """This norm and `other` (an RMS norm with the same eps) of the same stream, behind the pending term: two normed
+        tensors by one kernel."""
+        res = h if isinstance(h, Residual) else Residual(h)
+        if other.eps != self.eps:
+            raise ValueError("two norms of one stream in one kernel have the same eps")
+        if isinstance(delta, NormedTerm):
+            return step.ops.add_rmsnorm_pair(res.data, delta.data, self.weight, other.weight, self.eps, self.dtype, delta.gamma, delta.eps)
+        return step.ops.add_rmsnorm_pair(res.data, delta, self.weight, other.weight, self.eps, self.dtype)
+
+
 class LayerNorm(Norm):
     """`(x - mean) / sqrt(var + eps) * weight + bias` over the row, the variance being the mean of the squared
     deviations; all in 32-bit.  The pending term is added into the 32-bit residual stream by the same kernel."""

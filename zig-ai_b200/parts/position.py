@@ -37,6 +37,10 @@ class RotaryHalfSplit(PositionEncoding):
         rotation has none and is applied from `table`."""
         return (self.rotary_dim, self.theta) if self.scaling is None else None
 
+    def rotation(self):
+        """(rotary_dim, theta, scaling) for the kernels that take the table of a stretched rotation, too."""
+        return self.rotary_dim, self.theta, self.scaling
+
     def table(self, step, device):
         """(rotated dimensions, (cos, sin) per row of the step and pair [N, dims/2, 2] in 32-bit), made once per
         step and rotation."""
@@ -64,6 +68,9 @@ class NoPosition(PositionEncoding):
 
     def rotary(self):
         return 0, 1.0
+
+    def rotation(self):
+        return 0, 1.0, None
 
     def table(self, step, device):
         return 0, None
