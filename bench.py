@@ -254,6 +254,8 @@ def run_ours(args):
         return run_lolivik(args)
     if args.only == "sogenex":
         return run_sogenex(args)
+    if args.only == "pirozen":
+        return run_pirozen(args)
     if args.only == "long":
         return run_long(args)
     if args.only == "sample":
@@ -370,21 +372,26 @@ def vunolorn_config(width, layers=16, vocab=65536):
 
 
 def engine_numbers(eng):
-    """From the engine itself, for any architecture: matrix parameters a step reads, bytes of keys and values per
-    cached position, bytes of per-request state."""
-    decls = eng.runner.model.param_decls()
+    """From the engine itself, for any architecture: matrix parameters a step reads (of a layer that runs several times, in every
+    run), bytes of keys and values per cached position, bytes of per-request state."""
+    model = eng.runner.model
+    decls = model.param_decls()
     numel = lambda shape: int(__import__("math").prod(shape))
     matrix = sum(numel(d.shape) for d in decls.values() if d.role == "matrix")
+    runs = [sum(c.layer == i for c in model.spec.order) for i in range(len(model.blocks))]
+    for n, blk in zip(runs, model.blocks):
+        for part in [blk] + list(blk.parts().values()):
+            matrix += (n - 1) * sum(numel(d.shape) for d in part.params().values() if d.role == "matrix")
     if getattr(eng.runner.model.head, "tied", False):
         matrix += sum(numel(d.shape) for d in decls.values() if d.role == "table")
     cache = eng.runner.cache
     state = sum(len(g.members) * numel(g.need.shape) * 4 for g in cache.groups if not g.paged)
     routed = []        # (experts, experts a token uses, parameters of one expert) of every mixture of experts
-    for blk in eng.runner.model.blocks:
+    for blk in (model.blocks[c.layer] for c in model.spec.order):
         ff = getattr(blk, "feed_forward", None)
         if ff is not None and hasattr(ff, "experts") and hasattr(ff, "top"):
             per = 2 if getattr(ff, "expert_act", "") == "relu2" else 3            # matrices an expert has
-            routed.append((ff.experts, ff.top, per * ff.hidden * ff.ff_dim))
+            routed.append((ff.experts, ff.top * ff.experts / ff.outputs, per * ff.hidden * ff.ff_dim))
     return dict(matrix_params=matrix, kv_bytes_per_token=cache.bytes_per_token(), state_bytes=state, routed=routed)
 
 
@@ -1156,6 +1163,166 @@ def run_sogenex(args):
     return run_beside(args, lambda w: ((f"Sogenex-{w}", sogenex_config(w)), (f"Lolivik-{w}", lolivik_config(w))), sogenex_kernel_rooflines)
 
 
+def pirozen_config(width, layers=12, vocab=65536):
+    """A Pirozen model of a real model's proportions, run as sixteen layers: windowed attention (heads of 64, four query heads a
+    key/value head, a window of 1024, half of a head rotated) beside twelve experts and four identities in four groups, three
+    outputs a token out of two groups, and an expert for every token; side rows of width / 16 entries a layer; layers 4 to 7 run
+    twice."""
+    heads = width // 64
+    att = {"heads": heads, "kv_heads": heads // 4, "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": 1024},
+           "rot": {"base": 5e5, "dims": 32, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": width}, "router": {"experts": 12, "identity": 4, "top": 3, "scale": 1.5, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": width}}
+    return {"architecture": "Pirozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": width // 16},
+            "loop": {"start": 4, "stop": 8, "times": 2},
+            "layers": [{"type": "attention", "mixer": dict(att), "mlp": dict(moe)} for _ in range(layers)]}
+
+
+def pirozen_kernel_rooflines(width, hbm_peak, flops_peak):
+    """Every kernel that the design adds, alone at the sizes of `pirozen_config(width)`, beside the like kernel of an existing
+    design: the attention from the projection's rows to the output projection's input (norm, rotation, pages, windowed softmax,
+    gate), at equal sizes of keys and values and at keys of twice the values' size, beside Lolivik's windowed attention with its
+    preparation; the experts with identities, corrections and groups, combined onto the stream, beside Lolivik's bounded experts
+    with as many outputs a token that have matrices; the two norms beside one; the merge of stream and embedding and the products with a bias beside
+    plain products; the term from the side rows beside the two plain products of its size.  A portion of 2048 tokens and 64 and 8
+    single tokens over contexts of 2048, timed with CUDA events, the L2 flushed before every call; `distance` is the time over
+    the larger of the two roofline times."""
+    import torch
+    from zig_ai_b200.cache.manager import CacheView
+    from zig_ai_b200.engine.batch import pack_step
+    from zig_ai_b200.kernels import ops
+    from zig_ai_b200.parts import PartSpec, make_part
+    ops.require(torch.bfloat16, ("attention", "attention_mma", "attention_tma", "attention_tc", "qkv_prepare", "moe", "gemm_tc"))
+    dev, dt = torch.device("cuda"), torch.bfloat16
+    ps, E, I, top, F, side = 64, 12, 4, 3, width, width // 16
+    g = torch.Generator().manual_seed(1)
+    rnd = lambda *shape, s=1.0: (torch.randn(*shape, generator=g) * s).to(dt).to(dev)
+    rows = []
+
+    def step_of(ctx, q_lens):
+        spans, tables, at = [], [], 1
+        width_pages = max(-(-(c + n) // ps) for c, n in zip(ctx, q_lens))
+        for s_, (c, n) in enumerate(zip(ctx, q_lens)):
+            need = -(-(c + n) // ps)
+            tables.append(list(range(at, at + need)) + [0] * (width_pages - need))
+            at += need
+            spans.append((s_, c, [0] * n, [], s_ + 1))
+        return pack_step(ops, dt, dev, spans, {0: tables}), at
+
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=10):
+        for _ in range(3):
+            fn()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        total = 0.0
+        for _ in range(reps):
+            flush.zero_()                                    # larger than L2: the timed call starts cold
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            total += a.elapsed_time(b)
+        return total / reps
+
+    stretch = {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+
+    def attention(H, G, D, V, lolivik):
+        """The attention part without its two products: a part whose projections are not run, called from their rows on."""
+        position = PartSpec("rotary_interleaved" if lolivik else "rotary_half_split",
+                            dict(head_dim=D, theta=5e5, rotary_dim=D // 2, scaling=dict(kind="wavelength", factor=4.0, low=1.0, high=4.0, original=8192)
+                                 if lolivik else stretch))
+        more = dict(keep_first=4) if lolivik else dict(bias=True, out_bias=True, gate="head")
+        part = make_part("mixer", PartSpec("attention", dict(hidden=64, heads=H, kv_heads=G, head_dim=D, value_dim=V, qk_norm=True, eps=1e-6,
+                                                             position=position, window=1024, scale=0.125, **more)))
+        part.bind({n: (torch.ones(d.shape, device=dev) if d.role == "vector" else torch.zeros(d.shape, dtype=dt, device=dev))
+                   for n, d in part.params().items()}, dt)
+        return part
+
+    def rows_only(part, y, step, view):
+        class Ops:                                           # the kernels, with the part's products left out
+            def __getattr__(self, name):
+                return getattr(ops, name)
+
+            @staticmethod
+            def linear(x, w, bias=None):
+                return y if w is part.w_qkv else x
+        call = Ops()
+
+        def run():
+            keep, step.ops = step.ops, call
+            step.scratch.pop("attention.v_first", None)
+            part.forward(y, step, view)
+            step.ops = keep
+        return run
+
+    for point, ctx, q_lens in (("2048-token portion", [0], [2048]), ("64 single tokens, context 2048", [2047] * 64, [1] * 64),
+                               ("8 single tokens, context 2048", [2047] * 8, [1] * 8)):
+        step, n_pages = step_of(ctx, q_lens)
+        N, B = sum(q_lens), len(q_lens)
+        pairs = sum(sum(min(c + i + 1, 1024) for i in range(n)) for c, n in zip(ctx, q_lens))
+        cached = sum(min(c + n, 1023 + n) for c, n in zip(ctx, q_lens))
+        for H, D, V, lolivik, label in ((width // 64, 64, 64, False, "windowed attention with gate, heads of 64"),
+                                        (width // 128, 128, 64, False, "windowed attention with gate, keys of 128, values of 64"),
+                                        (width // 64, 64, 64, True, "windowed attention, first positions kept, heads of 64 (Lolivik's)"),
+                                        (width // 128, 128, 128, True, "windowed attention, first positions kept, heads of 128 (Lolivik's)")):
+            G = H // 4
+            part = attention(H, G, D, V, lolivik)
+            y = rnd(N, part.w_qkv.shape[0])
+            view = CacheView(0, rnd(n_pages, 2, G, ps, part.cache_dim, s=0.5), step.block_tables[0], ps)
+            rows.append((label, point, timed(rows_only(part, y, step, view)), 2.0 * pairs * H * (D + V), cached * G * (D + V) * 2 + N * H * (D + V) * 2))
+        # the feed-forwards: of a token's three outputs, nine quarters have matrices on average
+        x, h, m = rnd(N, width), torch.randn(N, width, generator=g).to(dev), rnd(N, width)
+        w_router, corr = (torch.randn(E + I, width, generator=g) * 0.05).to(dev), (torch.randn(E + I, generator=g) * 0.02).to(dev)
+        w_gu, w_dn = rnd(E, 2 * F, width, s=0.02), rnd(E, width, F, s=0.02)
+        u_gu, u_dn = rnd(2 * F, width, s=0.02), rnd(width, F, s=0.02)
+        unit = lambda: ops.linear(ops.linear_swiglu(x, u_gu, F), u_dn)
+        active = top * E / (E + I)
+        used = E * (1 - (1 - active / E) ** N)
+        fl, by = 2.0 * N * (active + 1) * 3 * width * F, (used + 1) * 3 * width * F * 2 + N * width * 12
+        rows.append((f"experts ({top} of {E} and {I} identities, groups) and their unit, onto the stream", point, timed(lambda: ops.routed_experts(
+            x, w_router, w_gu, w_dn, top, True, "output", score="softmax", unit=unit(), correction=corr, groups=(4, 2), identities=I, weight_scale=1.5,
+            onto=(h, m, True))), fl, by))
+        w12 = w_router[:E].contiguous()
+        fl2, by2 = 2.0 * N * (2 + 1) * 3 * width * F, (E * (1 - (1 - 2 / E) ** N) + 1) * 3 * width * F * 2 + N * width * 12
+        bounded = lambda: ops.weighted_sum(
+            ops.routed_experts(x, w12, w_gu, w_dn, 2, True, "output", score="softmax", act="clamped", limit=7.0, alpha=1.702),
+            ops.linear(ops.linear_clamped_glu(x, u_gu, F, 7.0, 1.702), u_dn), 1.0, 1.0)
+        w1, w2 = torch.ones(width, device=dev), torch.ones(width, device=dev)
+        rows.append((f"bounded experts (2 of {E}) and their unit, then onto the stream (Lolivik's)", point,
+                     timed(lambda: ops.add_cast(h, bounded(), dt, w1, 1e-6)), fl2, by2))
+        rows.append(("two norms of the stream and a normed term", point, timed(lambda: ops.add_rmsnorm_pair(h, m, w1, w2, 1e-6, dt, w1, 1e-6)), 0.0, N * width * 14))
+        rows.append(("one norm of the stream and a normed term (Lolivik's, Vunolorn's)", point, timed(lambda: ops.add_rmsnorm(h, m, w1, 1e-6, dt, w1, 1e-6)), 0.0,
+                     N * width * 12))
+        # products
+        O = (width // 64 + 2 * (width // 256)) * 64
+        w_q, b_q = rnd(O, width, s=0.02), rnd(O)
+        fl, by = 2.0 * N * O * width, O * width * 2 + N * (O + width) * 2
+        rows.append(("projection with a bias", point, timed(lambda: ops.linear(x, w_q, bias=b_q)), fl, by))
+        rows.append(("projection without (shared by all)", point, timed(lambda: ops.linear(x, w_q)), fl, by))
+        w_m, c_m = rnd(width, width, s=0.02), torch.randn(N, width, generator=g).to(dev)
+        fl, by = 2.0 * N * width * width, width * width * 2 + N * width * 10
+        rows.append(("merge: the stream's product and the embedding's share", point, timed(lambda: ops.linear_add(x, w_m, c_m)), fl, by))
+        rows.append(("the same product alone, 32-bit result (shared by all)", point, timed(lambda: ops.linear(x, w_m, out_dtype=torch.float32)), fl,
+                     by - N * width * 4))
+        w_g, w_p = rnd(side, width, s=0.02), rnd(width, side, s=0.02)
+        table, ids = rnd(65536, 12 * side), torch.randint(0, 65536, (N,), generator=g).to(torch.int32).to(dev)
+        fl, by = 4.0 * N * width * side, 2 * width * side * 2 + N * (2 * width + side) * 2
+        rows.append(("side rows: gate, lookup, projection", point, timed(lambda: ops.linear(ops.linear_side(x, w_g, table, ids, side), w_p)), fl, by))
+        rows.append(("two plain products of that size (shared by all)", point, timed(lambda: ops.linear(ops.linear(x, w_g), w_p)), fl, by - N * side * 2))
+    return [{"kernel": k, "point": p, "width": width, "us": round(ms * 1e3, 2), "GFLOP": round(fl / 1e9, 2), "MB": round(by / 1e6, 2),
+             "TFLOP_per_s": round(fl / ms / 1e9, 1), "of_tensor_peak": round(fl / ms / 1e9 / flops_peak, 4),
+             "GB_per_s": round(by / ms / 1e6, 1), "of_copy_peak": round(by / ms / 1e6 / hbm_peak, 4),
+             "distance": round(ms / max(fl / 1e9 / flops_peak, by / 1e6 / hbm_peak), 2)} for k, p, ms, fl, by in rows]
+
+
+def run_pirozen(args):
+    """Prefill and decode throughput of the Pirozen design at two widths beside the Lolivik design (the closest one: windowed
+    attention with a stretched rotation and experts by softmax score with a unit for every token) of the same width, layer runs
+    and vocabulary; the time of a prefill and of a decode step by kernel class; and its kernels alone beside the like kernels."""
+    return run_beside(args, lambda w: ((f"Pirozen-{w}", pirozen_config(w)), (f"Lolivik-{w}", lolivik_config(w))), pirozen_kernel_rooflines)
+
+
 def run_table(args):
     """The tracked table: the 350M, 700M and 1.2B shapes, decode at batch 1/8/64 device-timed and end to end,
     the prefill of 2048 tokens, and the mixed workload of the 700M shape, as JSON lines and as markdown."""
@@ -1509,9 +1676,9 @@ def main():
     ap.add_argument("--steps", type=int, default=200)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "gemm", "timeline", "table", "stream", "long", "sample", "vunolorn", "pikasun", "zikevik", "lolivik", "sogenex"],
+    ap.add_argument("--only", default="all", choices=["all", "decode", "prefill", "gemm", "timeline", "table", "stream", "long", "sample", "vunolorn", "pikasun", "zikevik", "lolivik", "sogenex", "pirozen"],
                     help="profiling aid: run only the batch-8 decode steps or only the prefill (prints a short line); "
-                         "table: every figure of the 350M, 700M and 1.2B shapes (profiles/measurements.md); pikasun: the Pikasun design beside LFM2 at equal width; zikevik: the Zikevik design beside Pikasun at equal width, and its kernels beside the like ones; lolivik: the Lolivik design beside Zikevik at equal width, and its kernels beside the like ones; sogenex: the Sogenex design beside Lolivik, likewise; vunolorn: the "
+                         "table: every figure of the 350M, 700M and 1.2B shapes (profiles/measurements.md); pikasun: the Pikasun design beside LFM2 at equal width; zikevik: the Zikevik design beside Pikasun at equal width, and its kernels beside the like ones; lolivik: the Lolivik design beside Zikevik at equal width, and its kernels beside the like ones; sogenex: the Sogenex design beside Lolivik, likewise; pirozen: the Pirozen design beside Lolivik, likewise; vunolorn: the "
                          "Vunolorn hybrid at two widths beside LFM2 at equal width, and its recurrent kernels alone")
     ap.add_argument("--batch", type=int, default=8, help="with --only decode: the batch size; with --only stream: 24, 64 or "
                                                          "128 runs that row count only")

@@ -557,7 +557,7 @@ template <int D> static size_t decode_smem();
 // kernel, the combine kernel; the reference has one kernel each for norm, rotary, append and
 // attention, src/transformer/hybrid_attn.zig:710-764).
 struct FusedDecodeArgs {
-    bf16* out;                 // [B, Hq, D]
+    bf16* out;                 // [B, Hq, out_dim]
     float* part_o;             // [B, Hq, n_chunks, D]
     float* part_ml;            // [B, Hq, n_chunks, 2]
     int* tickets;              // [B * Hkv], zero before and after
@@ -570,6 +570,8 @@ struct FusedDecodeArgs {
     const int* positions;
     float eps, scale_log2;
     int q_map;                 // > 0: the projection holds pairs of maps (query_head)
+    const bf16* gate;          // a number per query head in the rows of qkv: outputs times its sigmoid; or null
+    int out_dim;               // values of a head that are written (the first ones; the rest are zeros of narrower values)
     int qkv_cols, rot, table_width, page_size, Hq, Hkv, window, write_kv;
     int num_pages;             // pages in `pages`: a table entry outside is read as page 0 and raises the status word
     int* status;
@@ -797,6 +799,7 @@ __global__ void __launch_bounds__(NTHREADS) decode_fused_kernel(const FusedDecod
     __syncthreads();
     if (s_ticket != n_chunks - 1) return;
     __threadfence();
+    const bf16* gate = a.gate ? a.gate + (size_t)b * a.qkv_cols : nullptr;
     for (int idx = tid; idx < G * D; idx += NTHREADS) {
         const int r = idx / D, d = idx % D;
         const size_t bh = (size_t)b * Hq + hk * G + r;
@@ -811,7 +814,9 @@ __global__ void __launch_bounds__(NTHREADS) decode_fused_kernel(const FusedDecod
             acc += __ldcg(a.part_o + (bh * n_chunks + c) * D + d) * f;
             L += __ldcg(ml + 2 * c + 1) * f;
         }
-        a.out[bh * D + d] = __float2bfloat16_rn(acc / L);
+        float v = acc / L;
+        if (gate) v /= 1.f + expf(-__bfloat162float(gate[hk * G + r]));
+        if (d < a.out_dim) a.out[bh * a.out_dim + d] = __float2bfloat16_rn(v);
     }
     if (tid == 0) a.tickets[b * Hkv + hk] = 0;
 }
@@ -967,14 +972,16 @@ ZAI_API int zai_decode_attention_mma(void* out, float* part_o, float* part_ml, c
 
 // The decode step's attention from the raw qkv rows: see decode_fused_kernel.  `tickets` holds
 // B * Hkv zeros (and again after the call).  q_map > 0: the rows hold Hq / 2 query heads, each two maps of q_map and D - q_map
-// values, which count as two query heads with zeros in the other map's place (no norm, no rotation).
+// values, which count as two query heads with zeros in the other map's place (no norm, no rotation).  `gate` (or null): the
+// columns of qkv's rows that hold a number per query head whose sigmoid multiplies that head's output; out is [B, Hq, out_dim].
 ZAI_API int zai_decode_attention_fused(void* out, float* part_o, float* part_ml, int* tickets, const void* qkv,
                                        int qkv_cols, const float* q_gamma, const float* k_gamma, float eps,
                                        const float2* cs_table, int rot, void* pages, const int* block_table,
                                        int table_width, const int* positions, int B, int n_chunks, int page_size,
                                        int Hq, int Hkv, int D, float scale, int window, int write_kv, int chunk_keys,
-                                       int num_pages, int* status, int q_map, cudaStream_t stream) {
+                                       int num_pages, int* status, int q_map, const void* gate, int out_dim, cudaStream_t stream) {
     if (B <= 0) return ZAI_OK;
+    if (out_dim < 1 || out_dim > D) return ZAI_BAD_SIZE;
     if (q_map < 0 || q_map > D || (q_map && ((Hq & 1) || rot || q_gamma))) return ZAI_BAD_SIZE;
     if (chunk_keys < TILE || chunk_keys % TILE) return ZAI_BAD_SIZE;
     if (n_chunks < 1 || Hkv < 1 || Hkv > 65535 || B > 65535 || Hq % Hkv != 0 || Hq / Hkv > 16 || rot < 0 || rot > D || (rot & 1))
@@ -983,6 +990,7 @@ ZAI_API int zai_decode_attention_fused(void* out, float* part_o, float* part_ml,
     a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.tickets = tickets; a.qkv = (const bf16*)qkv;
     a.q_gamma = q_gamma; a.k_gamma = k_gamma; a.cs_table = cs_table; a.pages = (bf16*)pages; a.block_table = block_table;
     a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot; a.q_map = q_map;
+    a.gate = (const bf16*)gate; a.out_dim = out_dim;
     a.table_width = table_width; a.page_size = page_size; a.Hq = Hq; a.Hkv = Hkv; a.window = window; a.write_kv = write_kv; a.chunk_keys = chunk_keys;
     a.num_pages = num_pages; a.status = status;
 #define X(d) if (D == d) return launch_decode_fused<d>(a, B, n_chunks, stream);

@@ -81,7 +81,7 @@ __device__ __forceinline__ void pv_16keys_sw(float (&o)[TT_D / 8][4], const uint
 }
 
 struct TmaDecodeArgs {
-    bf16* out;                 // [B, Hq, 64]
+    bf16* out;                 // [B, Hq, out_dim]
     float* part_o;             // [B, Hq, n_chunks, 64]
     float* part_ml;            // [B, Hq, n_chunks, 2]
     int* tickets;              // [B * Hkv], zero before and after
@@ -96,6 +96,8 @@ struct TmaDecodeArgs {
     const int* positions;
     float eps, scale_log2;
     int q_map;                 // > 0: the projection holds pairs of maps (query_head)
+    const bf16* gate;          // a number per query head in the rows of qkv: outputs times its sigmoid; or null
+    int out_dim;               // values of a head that are written (the first ones; the rest are zeros of narrower values)
     int qkv_cols, rot, table_width, page_size, page_shift, Hq, Hkv, window, write_kv, chunk_keys, stages;
     int chunk_fastest;         // the grid is (chunks, Hkv, B) if set, else (Hkv, B, chunks)
 };
@@ -391,6 +393,7 @@ __global__ void __maxnreg__(128) decode_tma_kernel(const __grid_constant__ CUten
     __syncthreads();
     if (s_ticket != n_chunks - 1) return;
     __threadfence();
+    const bf16* gate = a.gate ? a.gate + (size_t)b * a.qkv_cols : nullptr;
     for (int idx = tid; idx < G * D; idx += TT_THREADS) {
         const int r = idx / D, d = idx % D;
         const size_t bh = (size_t)b * Hq + hk * G + r;
@@ -405,7 +408,9 @@ __global__ void __maxnreg__(128) decode_tma_kernel(const __grid_constant__ CUten
             acc += __ldcg(a.part_o + (bh * n_chunks + c) * D + d) * f;
             L += __ldcg(ml + 2 * c + 1) * f;
         }
-        a.out[bh * D + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+        float v = L > 0.f ? acc / L : 0.f;
+        if (gate) v /= 1.f + expf(-__bfloat162float(gate[hk * G + r]));
+        if (d < a.out_dim) a.out[bh * a.out_dim + d] = __float2bfloat16_rn(v);
     }
     if (tid == 0) a.tickets[b * Hkv + hk] = 0;
 }
@@ -452,8 +457,9 @@ ZAI_API int zai_decode_attention_tma(void* out, float* part_o, float* part_ml, i
                                      const float2* cs_table, int rot, void* pages, int num_pages, const int* block_table,
                                      int table_width, const int* positions, int B, int n_chunks, int page_size, int Hq,
                                      int Hkv, int D, float scale, int window, int write_kv, int chunk_keys,
-                                     int q_map, cudaStream_t stream) {
+                                     int q_map, const void* gate, int out_dim, cudaStream_t stream) {
     if (B <= 0) return ZAI_OK;
+    if (out_dim < 1 || out_dim > D) return ZAI_BAD_SIZE;
     if (q_map < 0 || q_map > D || (q_map && ((Hq & 1) || rot || q_gamma))) return ZAI_BAD_SIZE;
     if (!zai_decode_attention_tma_supports(D, Hq, Hkv, page_size)) return ZAI_BAD_SIZE;
     if (chunk_keys < TT_TILE || chunk_keys % TT_TILE || n_chunks < 1 || Hkv > 65535 || B > 65535 || n_chunks > 65535 || rot < 0 || rot > D || (rot & 1))
@@ -472,6 +478,7 @@ ZAI_API int zai_decode_attention_tma(void* out, float* part_o, float* part_ml, i
     a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.tickets = tickets; a.status = status; a.num_pages = num_pages; a.qkv = (const bf16*)qkv;
     a.q_gamma = q_gamma; a.k_gamma = k_gamma; a.cs_table = cs_table; a.pages = (bf16*)pages; a.block_table = block_table;
     a.positions = positions; a.eps = eps; a.scale_log2 = scale * 1.4426950408889634f; a.qkv_cols = qkv_cols; a.rot = rot; a.q_map = q_map;
+    a.gate = (const bf16*)gate; a.out_dim = out_dim;
     a.table_width = table_width; a.page_size = page_size; a.Hq = Hq; a.Hkv = Hkv; a.window = window; a.write_kv = write_kv;
     a.chunk_keys = chunk_keys;
     a.page_shift = 0;

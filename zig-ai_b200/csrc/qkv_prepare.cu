@@ -97,6 +97,96 @@ __global__ void __launch_bounds__(256) qkv_prepare_kernel(
     }
 }
 
+// The same work for bfloat16 heads of multiples of eight values (norm per head or none): eight lanes' worth of a head's row a
+// time, `lanes` (a power of two) neighbouring lanes a head, eight values a lane, each in registers from the projection's row to
+// the page; a row's heads of q, k and v are independent items.  A rotated pair's other half comes from the lane that holds it.
+__device__ __forceinline__ void prep_load8(float (&v)[8], const bf16* p) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        v[2 * i] = f.x; v[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ void prep_store8(bf16* p, const float (&v)[8]) {
+    uint4 u;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = u;
+}
+__global__ void __launch_bounds__(256) qkv_prepare_heads_kernel(
+    const bf16* __restrict__ y, int y_stride, const float* __restrict__ q_gamma, const float* __restrict__ k_gamma, float eps,
+    const float2* __restrict__ cs_table, int rot, const int* __restrict__ positions, const int* __restrict__ seq_idx,
+    const int* __restrict__ block_table, int table_width, bf16* __restrict__ pages, int page_size, bf16* __restrict__ q_out, int N,
+    int Hq, int Hkv, int D, int Dv, int Dp, int write, int num_pages, int* __restrict__ status, float temp_coef, int temp_every,
+    const bf16* __restrict__ v_first, int v_first_stride, const float* __restrict__ v_lambda, int lanes) {
+    pdl_trigger();
+    pdl_wait();
+    const unsigned heads = Hq + (write ? 2 * Hkv : 0), per_block = blockDim.x / lanes;
+    const unsigned item = blockIdx.x * per_block + threadIdx.x / lanes;
+    const bool live = item < (unsigned)N * heads;                        // (whole groups of lanes; all lanes stay for the exchanges)
+    const unsigned t = live ? item / heads : 0, hh = live ? item - t * heads : 0;
+    const int sub = threadIdx.x & (lanes - 1), d = sub * 8, half = rot / 2;
+    const int kind = hh < (unsigned)Hq ? 0 : hh < (unsigned)(Hq + Hkv) ? 1 : 2, h = hh - (kind == 0 ? 0 : kind == 1 ? Hq : Hq + Hkv);
+    const int own = kind == 2 ? Dv : D;
+    const bf16* src = y + (size_t)t * y_stride + (kind == 0 ? (size_t)h * D : (size_t)Hq * D + (kind == 1 ? (size_t)h * D : (size_t)Hkv * D + (size_t)h * Dv));
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    const bool mine = live && d < own;
+    if (mine) prep_load8(v, src + d);
+    const int pos = positions[t];
+    const float* gamma = kind == 0 ? q_gamma : k_gamma;
+    if (gamma) {                                                         // (uniform over the launch; values' lanes discard it)
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
+        for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (mine && kind != 2) {
+            const float inv = rsqrtf(ss / (float)D + eps);
+            const float4 ga = *reinterpret_cast<const float4*>(gamma + d), gb = *reinterpret_cast<const float4*>(gamma + d + 4);
+            v[0] *= inv * ga.x; v[1] *= inv * ga.y; v[2] *= inv * ga.z; v[3] *= inv * ga.w;
+            v[4] *= inv * gb.x; v[5] *= inv * gb.y; v[6] *= inv * gb.z; v[7] *= inv * gb.w;
+        }
+    }
+    if (rot) {
+        const bool low = d < half;
+        const int base = (threadIdx.x & 31) & ~(lanes - 1), other = base + ((sub + (low ? half / 8 : -(half / 8))) & (lanes - 1));
+        float w[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) w[i] = __shfl_sync(0xffffffffu, v[i], other);
+        if (mine && kind != 2 && d < rot) {
+            const float2* cs = cs_table + (size_t)t * half + (low ? d : d - half);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float2 c = cs[i];
+                v[i] = low ? v[i] * c.x - w[i] * c.y : w[i] * c.y + v[i] * c.x;
+            }
+        }
+    }
+    if (!live || d >= Dp) return;
+    if (kind == 0) {
+        if (temp_every > 0) {
+            const float temp = 1.f + temp_coef * logf((float)((pos < 0 ? 0 : pos + 1) / temp_every + 1));
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] *= temp;
+        }
+        prep_store8(q_out + ((size_t)t * Hq + h) * Dp + d, v);
+        return;
+    }
+    if (kind == 2 && v_first && mine) {
+        float f[8];
+        prep_load8(f, v_first + (size_t)t * v_first_stride + (size_t)h * Dv + d);
+        const float lam = v_lambda[0];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = (1.f - lam) * v[i] + lam * f[i];
+    }
+    const int page = zai_checked_page(block_table + (size_t)seq_idx[t] * table_width, table_width, pos < 0 ? -1 : pos / page_size, num_pages,
+                                      status);
+    const int off = pos < 0 ? 0 : pos % page_size;
+    prep_store8(pages + (((size_t)page * 2 * Hkv + (kind == 1 ? 0 : Hkv) + h) * page_size + off) * Dp + d, v);
+}
+
 ZAI_API int zai_qkv_prepare(const void* y, int y_stride, int dtype, const float* q_gamma, const float* k_gamma, float eps, int scope,
                             const float2* cs_table, int rot, const int* positions, const int* seq_idx, const int* block_table,
                             int table_width, void* pages, int page_size, void* q_out, int N, int Hq, int Hkv, int D, int Dv,
@@ -106,6 +196,19 @@ ZAI_API int zai_qkv_prepare(const void* y, int y_stride, int dtype, const float*
     if (Hq < 1 || Hkv < 1 || D < 1 || Dv < 1 || Dp < D || Dp < Dv || rot < 0 || rot > D || rot % 2 || scope < 0 || scope > 2
         || (scope && (!q_gamma || !k_gamma)) || (rot && !cs_table) || temp_every < 0 || (v_first && !v_lambda))
         return ZAI_BAD_SIZE;
+    const uintptr_t at = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(q_out) |
+                         reinterpret_cast<uintptr_t>(v_first) | reinterpret_cast<uintptr_t>(q_gamma) | reinterpret_cast<uintptr_t>(k_gamma);
+    if (dtype == ZAI_BF16 && scope < 2 && ((D | Dv | Dp | y_stride | v_first_stride) & 7) == 0 && rot % 16 == 0 && Dp <= 256 && (at & 15) == 0
+        && (long long)N * (Hq + 2 * Hkv) < (1 << 30)) {
+        int lanes = 1;
+        while (lanes * 8 < Dp) lanes *= 2;
+        const long long items = (long long)N * (Hq + (write ? 2 * Hkv : 0));
+        const int per_block = 256 / lanes;
+        return launch_pdl(qkv_prepare_heads_kernel, dim3((unsigned)((items + per_block - 1) / per_block)), dim3(256), 0, stream, (const bf16*)y,
+                          y_stride, scope ? q_gamma : nullptr, scope ? k_gamma : nullptr, eps, cs_table, rot, positions, seq_idx, block_table,
+                          table_width, (bf16*)pages, page_size, (bf16*)q_out, N, Hq, Hkv, D, Dv, Dp, write, num_pages, status, temp_coef,
+                          temp_every, (const bf16*)v_first, v_first_stride, v_lambda, lanes);
+    }
     const size_t smem = ((size_t)(Hq + Hkv) * D + rot) * sizeof(float);
     if (smem > 200 * 1024) return ZAI_BAD_SIZE;
     static unsigned long long done_f32 = 0, done_bf16 = 0;

@@ -105,7 +105,7 @@ _SIGNATURES = {
         "zai_decode_attention_mma_scored": [_P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _P, _I, _P, _I,
                                             _P],
         "zai_decode_attention_fused": [_P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _I, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I,
-                                       _F, _I, _I, _I, _I, _P, _I, _P],
+                                       _F, _I, _I, _I, _I, _P, _I, _P, _I, _P],
         "zai_decode_chunk_keys": [],
         "zai_prefill_block_rows": [],
     },
@@ -140,7 +140,7 @@ _SIGNATURES = {
     "attention_tma": {
         "zai_decode_attention_tma_supports": [_I, _I, _I, _I],
         "zai_decode_attention_tma": [_P, _P, _P, _P, _P, _P, _I, _P, _P, _F, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I,
-                                     _I, _F, _I, _I, _I, _I, _P],
+                                     _I, _F, _I, _I, _I, _I, _P, _I, _P],
     },
     "attention_tc": {
         "zai_prefill_attention_tc_supports": [_I, _I, _I, _I],
@@ -1113,19 +1113,25 @@ def fused_decode_attention_available(dtype, heads, kv_heads, head_dim) -> bool:
 
 @_timed("attention (with q/k norm, rotation, page write)")
 def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, heads, kv_heads, head_dim, scale,
-                           window=None, write=True, q_map=0, scaling=None):
+                           window=None, write=True, q_map=0, scaling=None, gate_at=None, value_dim=None):
     """A decode step's attention in one kernel, from the qkv projection's rows [B, (Hq + 2 Hkv) D]:
     q/k RMSNorm, rotation, the new key and value into their page, attention over the pages in chunks
     of keys, and the combination of the chunks.  Every row of the step is one token.  `q_map`: as in `qk_norm_rope`;
-    `scaling`: of the rotation, as in `inverse_frequencies`."""
+    `scaling`: of the rotation, as in `inverse_frequencies`.  `gate_at`: the first of `heads` columns of qkv that hold a number
+    per head, whose sigmoid multiplies the head's output.  `value_dim`: only that many values of a head are returned (the rest
+    are zeros behind narrower values), [B, heads * value_dim]."""
     _cuda(qkv, q_w, k_w)
     B, cols = qkv.shape
+    value_dim = head_dim if value_dim is None else int(value_dim)
+    if gate_at is not None and int(gate_at) + heads > cols:
+        raise KernelError("decode_attention_fused: the rows do not hold the gates")
+    gate = None if gate_at is None else qkv.data_ptr() + int(gate_at) * qkv.element_size()
     if cols < ((heads // 2 if q_map else heads) + 2 * kv_heads) * head_dim:
         raise KernelError("decode_attention_fused: the rows do not hold the heads")
     if B != step.n_tokens:
         raise KernelError(f"{B} rows for a step of {step.n_tokens} rows")
     dev = qkv.device
-    out = torch.empty((B, heads * head_dim), dtype=qkv.dtype, device=dev)
+    out = torch.empty((B, heads * value_dim), dtype=qkv.dtype, device=dev)
     # keys per block: about DECODE_BLOCKS_WANTED blocks (a little more than the SMs hold at once), so
     # that a block's start-up and its partial sums are spread over many keys without leaving SMs
     # idle (a power of two between 256 and 1024)
@@ -1148,13 +1154,13 @@ def decode_attention_fused(qkv, q_w, k_w, eps, rotary_dim, theta, step, cache, h
             _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _status_ptr(dev), _ptr(qkv), cols, _ptr(q_w), _ptr(k_w),
             float(eps), _ptr(table), int(rotary_dim), _ptr(cache.pages), cache.pages.shape[0], _ptr(bt), bt.shape[1],
             _ptr(step.positions), B, n_chunks, cache.page_size, heads, kv_heads, head_dim, float(scale), int(window or 0),
-            int(bool(write)), chunk, int(q_map), _stream()), "decode_attention_tma")
+            int(bool(write)), chunk, int(q_map), gate, value_dim, _stream()), "decode_attention_tma")
         return out
     _check(_fn("attention_mma", "zai_decode_attention_fused")(
         _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _ptr(qkv), cols, _ptr(q_w), _ptr(k_w), float(eps),
         _ptr(table), int(rotary_dim), _ptr(cache.pages), _ptr(bt), bt.shape[1], _ptr(step.positions), B, n_chunks,
         cache.page_size, heads, kv_heads, head_dim, float(scale), int(window or 0), int(bool(write)), chunk,
-        cache.pages.shape[0], _status_ptr(dev), int(q_map), _stream()), "decode_attention_fused")
+        cache.pages.shape[0], _status_ptr(dev), int(q_map), gate, value_dim, _stream()), "decode_attention_fused")
     return out
 
 

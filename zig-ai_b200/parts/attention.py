@@ -242,11 +242,12 @@ class Attention(Mixer):
         y = ops.linear(x, self.w_qkv, bias=self.b_qkv)
         fused = getattr(ops, "fused_decode_attention_available", None)
         if self.one_kernel_decode and step.decode_only and fused is not None and fused(y.dtype, H, G, Dp):
-            # norm, rotation, page write, attention and the combination of the key ranges in one kernel
+            # norm, rotation, page write, attention, the combination of the key ranges and the gate in one kernel
             rot = self.position.rotation()
+            gated = dict(gate_at=self.gate_at, value_dim=Dv) if self.gate else {}
             o = ops.decode_attention_fused(y, self.q_norm, self.k_norm, self.norm_eps, rot[0], rot[1], step, cache, H, G, Dp, self.scale,
-                                           self.window, write_cache, scaling=rot[2])
-            return self._prepared_output(o, y, ops)
+                                           self.window, write_cache, scaling=rot[2], **gated)
+            return ops.linear(o, self.w_o, bias=self.b_o)
         dims, table = self.position.table(step, y.device)
         scope = 0 if not self.qk_norm else (2 if self.norm_scope == "whole" else 1)
         more = {}
@@ -265,11 +266,8 @@ class Attention(Mixer):
                                     sink=self.sink_w, keep_first=self.keep_first)
         else:
             o = ops.paged_attention(q, step, cache, H, G, Dp, self.scale, self.window, chunk=self.chunk)
-        return self._prepared_output(o, y, ops)
-
-    def _prepared_output(self, o, y, ops):
         if self.gate:
-            o = ops.sigmoid_gate(o, y[:, self.gate_at:self.gate_at + self.heads], self.heads, self.value_dim, True, row_dim=self.cache_dim)
+            o = ops.sigmoid_gate(o, y[:, self.gate_at:self.gate_at + H], H, Dv, True, row_dim=Dp)
         return ops.linear(o, self.w_o, bias=self.b_o)
 
     def bind(self, tensors, dtype):
